@@ -653,6 +653,14 @@ class PuzonexModel(FosovikModel):
     entry points and engine options as `FosovikModel`."""
 
 
+class SuvapelModel(FosovikModel):
+    """A layer-list decoder ("architecture": "Suvapel"): each layer one Dynamic-Tanh norm feeding a mixer and a SiLU-gated feed-forward
+    with biases whose outputs join the stream together, then a gated, RMS-normed row of the token's own embedding for the layer.
+    Mixers: the gated delta rule (short convolutions, unit keys and queries, an f32 matrix state per head), or sliding-window attention
+    with kept first tokens, convolved projections, a YaRN-scaled rotation and one gate per head beside a delta rule with a decay per key
+    channel.  Same entry points and engine options as `FosovikModel`."""
+
+
 # config.json -> model class, as `model_factory::create_backend` picks a backend by architecture (crane-serve/src/engine/model_factory.rs:471-560)
 def model_class(config: dict):
     if config.get("architecture") == "Fosovik":
@@ -663,6 +671,8 @@ def model_class(config: dict):
         return NifaraxModel
     if config.get("architecture") == "Puzonex":
         return PuzonexModel
+    if config.get("architecture") == "Suvapel":
+        return SuvapelModel
     if "talker_config" in config:
         return Qwen3TTSModel
     if "vision_config" in config:

@@ -202,7 +202,8 @@ gemv_kernel(GemvArgs a) {
 #pragma unroll
             for (int b = 0; b < B; ++b) {
                 const float r = NORM ? rstd_s[b] : 1.f;
-                const float g = acc_s[(size_t)b * rpc + 2 * u] * r, up = acc_s[(size_t)b * rpc + 2 * u + 1] * r;
+                float g = acc_s[(size_t)b * rpc + 2 * u] * r, up = acc_s[(size_t)b * rpc + 2 * u + 1] * r;
+                if (a.bias) { g += a.bias[r0 + 2 * u]; up += a.bias[r0 + 2 * u + 1]; }
                 a.y[(size_t)b * a.ldy + (r0 / 2 + u)] = glu_pair_f(g, up, a.glu_limit);
             }
         }
@@ -213,7 +214,8 @@ gemv_kernel(GemvArgs a) {
                 const float v = acc_s[(size_t)b * rpc + i] * (NORM ? rstd_s[b] : 1.f);
                 float* yp = a.y + (size_t)b * a.ldy + r0 + i;
                 if constexpr (EPI == GEMV_RESID) {
-                    float add = a.out_scale ? a.out_scale[r0 + i] * v : v;
+                    float add = a.bias ? v + a.bias[r0 + i] : v;
+                    if (a.out_scale) add *= a.out_scale[r0 + i];
                     if (a.gate) add *= 1.f / (1.f + expf(-(a.gate[(size_t)b * a.ldg + r0 + i] + (a.gate_bias ? a.gate_bias[r0 + i] : 0.f))));
                     *yp += add;
                 } else *yp = v;

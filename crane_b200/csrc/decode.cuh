@@ -64,6 +64,7 @@ struct GemvArgs {
     const float* gate;      // GEMV_RESID, nullable [B, ldg]: the added value is multiplied by sigmoid(gate[b, n] + gate_bias[n]) (gate_bias nullable)
     int ldg;
     const float* gate_bias;
+    const float* bias;      // GEMV_RESID / GEMV_SILU_MUL, nullable [N]: added to W x before out_scale / before the gated unit (rows interleaved like W's)
     const uint32_t* force_tokens;  // optional [out_stride]: teacher forcing -- token fed back at step s is force_tokens[s] (argmax still reported)
 };
 

@@ -229,18 +229,21 @@ template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile(
 // SPLIT: q, k, v (and the probabilities) are hi + lo bf16 pairs; every product keeps its three leading terms
 //   S = qh.kh + qh.kl + ql.kh          O += ph.vh + ph.vl + pl.vh
 // so the result carries ~16 mantissa bits instead of 8 (the f32-oracle parity mode; 3x the tensor work of 4 % of the flops).
-template <int D, bool CAUSAL, bool PAGED, bool SPLIT>
-__global__ void __launch_bounds__(256, D == 64 ? 2 : 1)
+template <int D, int DV, bool CAUSAL, bool PAGED, bool SPLIT>
+__global__ void __launch_bounds__(256, D == 64 && DV == 64 ? 2 : 1)
 flash_prefill_kernel(FlashArgs a) {
     pdl_wait();
     pdl_launch_dependents();
     constexpr int BM = 64;
-    constexpr int BN = (SPLIT || D > 128) ? 32 : 64;     // half-page key tiles wherever a 64-key tile x 2 groups x 2 stages would not fit
-    constexpr int STG = (SPLIT && D > 128) ? 1 : 2;      // stages per group (D = 256 with hi + lo planes: one)
+    constexpr int DM = D > DV ? D : DV;
+    constexpr int BN = (SPLIT || DM > 128) ? 32 : 64;     // half-page key tiles wherever a 64-key tile x 2 groups x 2 stages would not fit
+    constexpr int STG = (SPLIT && DM > 128) ? 1 : 2;      // stages per group (D = 256 with hi + lo planes: one)
     constexpr int LDS = D + 8;                 // padded row (elements): conflict-free ldmatrix
-    constexpr int TILE = BN * LDS;             // elements per K or V tile plane
-    constexpr int CPR = D / 8;                 // 16-byte chunks per row
+    constexpr int LDV = DV + 8;
+    constexpr int TILE = BN * LDS, TILEV = BN * LDV;      // elements per K / V tile plane
+    constexpr int CPR = D / 8, CPV = DV / 8;   // 16-byte chunks per K / V row
     constexpr int P = SPLIT ? 2 : 1;           // planes per operand
+    constexpr int STAGE = P * (TILE + TILEV);  // K hi | K lo | V hi | V lo
     extern __shared__ __align__(16) unsigned char fsm[];
     bf16* q_s = reinterpret_cast<bf16*>(fsm);  // [P][BM x LDS]
     bf16* kv_s = q_s + P * BM * LDS;           // [2 groups][STG][K hi | K lo | V hi | V lo]
@@ -272,9 +275,25 @@ flash_prefill_kernel(FlashArgs a) {
         if (SPLIT) cp_async16(smem_u32(q_s + BM * LDS + r * LDS + ch * 8), src + a.q_lo_off, qr < S ? 16 : 0);
     }
     auto load_kv = [&](int tile, int stage) {
-        bf16* ks = kv_s + (grp * STG + stage) * 2 * P * TILE;
+        bf16* ks = kv_s + (grp * STG + stage) * STAGE;
         bf16* vs = ks + P * TILE;
         const int kv0 = tile * BN;
+        if constexpr (D != DV) {                          // (paged launches only)
+            const size_t base = ((size_t)btab[kv0 / KV_PAGE] * a.nkv + kvh) * KV_PAGE + (kv0 % KV_PAGE);
+            for (int c = gtid; c < BN * CPR; c += 128) {
+                const int r = c / CPR, ch = c % CPR, sz = kv0 + r < T ? 16 : 0;
+                const bf16* src = a.k_pool + (base + r) * D + ch * 8;
+                cp_async16(smem_u32(ks + r * LDS + ch * 8), src, sz);
+                if (SPLIT) cp_async16(smem_u32(ks + TILE + r * LDS + ch * 8), src + a.kv_lo_off, sz);
+            }
+            for (int c = gtid; c < BN * CPV; c += 128) {
+                const int r = c / CPV, ch = c % CPV, sz = kv0 + r < T ? 16 : 0;
+                const bf16* src = a.v_pool + (base + r) * DV + ch * 8;
+                cp_async16(smem_u32(vs + r * LDV + ch * 8), src, sz);
+                if (SPLIT) cp_async16(smem_u32(vs + TILEV + r * LDV + ch * 8), src + a.kv_lo_off, sz);
+            }
+            return;
+        }
         for (int c = gtid; c < BN * CPR; c += 128) {
             const int r = c / CPR, ch = c % CPR;
             const int t = kv0 + r;
@@ -301,9 +320,9 @@ flash_prefill_kernel(FlashArgs a) {
     __syncthreads();                           // the Q tile is complete for both groups
     auto group_sync = [&]() { asm volatile("bar.sync %0, 128;" ::"r"(1 + grp) : "memory"); };
 
-    float o_acc[D / 8][4];
+    float o_acc[DV / 8][4];
 #pragma unroll
-    for (int i = 0; i < D / 8; ++i) { o_acc[i][0] = o_acc[i][1] = o_acc[i][2] = o_acc[i][3] = 0.f; }
+    for (int i = 0; i < DV / 8; ++i) { o_acc[i][0] = o_acc[i][1] = o_acc[i][2] = o_acc[i][3] = 0.f; }
     float m_row[2] = {-INFINITY, -INFINITY}, l_row[2] = {0.f, 0.f};
     const float sl2 = a.scale * 1.4426950408889634f;
     const bool mods = CAUSAL && (a.softcap > 0.f || a.dist_r1 || a.dist_table);
@@ -313,13 +332,16 @@ flash_prefill_kernel(FlashArgs a) {
     uint32_t qf[SPLIT ? 1 : D / 16][4];        // plain mode keeps the Q fragments in registers; SPLIT re-reads them from smem
 
     bool first = true;
-    if (t_first + grp < n_tiles) load_kv(t_first + grp, 0);
+    // the tiles of the kept first keys that the window does not reach come first, then the window's own
+    const int keep = (CAUSAL && a.window > 0) ? a.keep_first : 0, n_keep = min((keep + BN - 1) / BN, t_first), n_walk = n_keep + n_tiles - t_first;
+    auto tile_at = [&](int i) { return i < n_keep ? i : t_first + i - n_keep; };
+    if (grp < n_walk) load_kv(tile_at(grp), 0);
     cp_async_commit();
     int it = 0;
-    for (int tile = t_first + grp; tile < n_tiles; tile += 2, ++it) {
-        const int stage = STG == 2 ? (it & 1) : 0;
+    for (int ti = grp; ti < n_walk; ti += 2, ++it) {
+        const int tile = tile_at(ti), stage = STG == 2 ? (it & 1) : 0;
         if (STG == 2) {
-            if (tile + 2 < n_tiles) load_kv(tile + 2, stage ^ 1);
+            if (ti + 2 < n_walk) load_kv(tile_at(ti + 2), stage ^ 1);
             cp_async_commit();
             cp_async_wait<1>();
         } else {
@@ -334,7 +356,7 @@ flash_prefill_kernel(FlashArgs a) {
                 ldmatrix_x4(qf[SPLIT ? 0 : kk][0], qf[SPLIT ? 0 : kk][1], qf[SPLIT ? 0 : kk][2], qf[SPLIT ? 0 : kk][3], smem_u32(q_s + r * LDS + c));
             }
         }
-        const bf16* ks = kv_s + (grp * STG + stage) * 2 * P * TILE;
+        const bf16* ks = kv_s + (grp * STG + stage) * STAGE;
         const bf16* vs = ks + P * TILE;
         // ---- S = Q K^T ----
         float s_acc[BN / 8][4];
@@ -390,7 +412,7 @@ flash_prefill_kernel(FlashArgs a) {
             for (int e = 0; e < 4; ++e) {
                 const int col = kv0 + j * 8 + tq * 2 + (e & 1);
                 const int qrow = q0 + warp * 16 + g + (e >> 1) * 8;
-                const bool vis = (col < T) && (!CAUSAL || (col <= kv_off + qrow && (a.window <= 0 || kv_off + qrow - col < a.window)));
+                const bool vis = (col < T) && (!CAUSAL || (col <= kv_off + qrow && (a.window <= 0 || kv_off + qrow - col < a.window || col < keep)));
                 float v = vis ? s_acc[j][e] * sl2 : -INFINITY;
                 if (CAUSAL && mods && vis) {          // cap, then the distance terms, in f32 on the scaled score
                     float sc = s_acc[j][e] * a.scale;
@@ -431,7 +453,7 @@ flash_prefill_kernel(FlashArgs a) {
         l_row[0] += ps[0];
         l_row[1] += ps[1];
 #pragma unroll
-        for (int i = 0; i < D / 8; ++i) {
+        for (int i = 0; i < DV / 8; ++i) {
             o_acc[i][0] *= corr[0]; o_acc[i][1] *= corr[0];
             o_acc[i][2] *= corr[1]; o_acc[i][3] *= corr[1];
         }
@@ -444,14 +466,14 @@ flash_prefill_kernel(FlashArgs a) {
             split_bf16x2(s_acc[2 * kt + 1][0], s_acc[2 * kt + 1][1], pa[2], pl[2]);
             split_bf16x2(s_acc[2 * kt + 1][2], s_acc[2 * kt + 1][3], pa[3], pl[3]);
 #pragma unroll
-            for (int dj = 0; dj < D / 8; dj += 2) {
+            for (int dj = 0; dj < DV / 8; dj += 2) {
                 uint32_t b0, b1, b2, b3;
                 const int r = kt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
                 const int c = dj * 8 + (lane >> 4) * 8;
-                ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(vs + r * LDS + c));
+                ldmatrix_x4_trans(b0, b1, b2, b3, smem_u32(vs + r * LDV + c));
                 if constexpr (SPLIT) {
                     uint32_t c0, c1, c2, c3;
-                    ldmatrix_x4_trans(c0, c1, c2, c3, smem_u32(vs + TILE + r * LDS + c));
+                    ldmatrix_x4_trans(c0, c1, c2, c3, smem_u32(vs + TILEV + r * LDV + c));
                     mma_bf16_16816(o_acc[dj], pl, b0, b1);
                     mma_bf16_16816(o_acc[dj + 1], pl, b2, b3);
                     mma_bf16_16816(o_acc[dj], pa, c0, c1);
@@ -463,32 +485,32 @@ flash_prefill_kernel(FlashArgs a) {
         }
         first = false;
         group_sync();      // the group is done with this stage before it is refilled
-        if (STG == 1 && tile + 2 < n_tiles) { load_kv(tile + 2, 0); cp_async_commit(); }
+        if (STG == 1 && ti + 2 < n_walk) { load_kv(tile_at(ti + 2), 0); cp_async_commit(); }
     }
     cp_async_wait<0>();
     // ---- merge the two groups' states (group 1 -> group 0 through its own, now idle, tile buffer) ----
     {
-        float* mg = reinterpret_cast<float*>(kv_s + STG * 2 * P * TILE);        // group 1's ring: [128 threads][D / 2 + 4] floats
-        constexpr int MW = D / 2 + 4;
+        float* mg = reinterpret_cast<float*>(kv_s + STG * STAGE);        // group 1's ring: [128 threads][DV / 2 + 4] floats
+        constexpr int MW = DV / 2 + 4;
         __syncthreads();
         if (grp == 1) {
             float* d = mg + (size_t)gtid * MW;
 #pragma unroll
-            for (int i = 0; i < D / 8; ++i) { d[4 * i] = o_acc[i][0]; d[4 * i + 1] = o_acc[i][1]; d[4 * i + 2] = o_acc[i][2]; d[4 * i + 3] = o_acc[i][3]; }
-            d[D / 2] = m_row[0]; d[D / 2 + 1] = m_row[1]; d[D / 2 + 2] = l_row[0]; d[D / 2 + 3] = l_row[1];
+            for (int i = 0; i < DV / 8; ++i) { d[4 * i] = o_acc[i][0]; d[4 * i + 1] = o_acc[i][1]; d[4 * i + 2] = o_acc[i][2]; d[4 * i + 3] = o_acc[i][3]; }
+            d[DV / 2] = m_row[0]; d[DV / 2 + 1] = m_row[1]; d[DV / 2 + 2] = l_row[0]; d[DV / 2 + 3] = l_row[1];
         }
         __syncthreads();
         if (grp == 1) return;
         const float* d = mg + (size_t)gtid * MW;
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
-            const float mo = d[D / 2 + r], lo = d[D / 2 + 2 + r];
+            const float mo = d[DV / 2 + r], lo = d[DV / 2 + 2 + r];
             const float mn = fmaxf(m_row[r], mo);
             const float c0 = (m_row[r] == -INFINITY) ? 0.f : exp2f(m_row[r] - mn), c1 = (mo == -INFINITY) ? 0.f : exp2f(mo - mn);
             m_row[r] = mn;
             l_row[r] = l_row[r] * c0 + lo * c1;
 #pragma unroll
-            for (int i = 0; i < D / 8; ++i) {
+            for (int i = 0; i < DV / 8; ++i) {
                 o_acc[i][2 * r] = o_acc[i][2 * r] * c0 + d[4 * i + 2 * r] * c1;
                 o_acc[i][2 * r + 1] = o_acc[i][2 * r + 1] * c0 + d[4 * i + 2 * r + 1] * c1;
             }
@@ -510,10 +532,12 @@ flash_prefill_kernel(FlashArgs a) {
                 const float c = exp2f(m_row[r] - mn);
                 inv = c / (l_row[r] * c + exp2f(s2 - mn));
             }
-            bf16* o = a.out + (size_t)(row0 + qrow) * a.o_stride + head * D;
-            const float* gt = a.gate ? a.gate + (size_t)(row0 + qrow) * a.g_stride + head * D : nullptr;
+            inv *= a.out_mult;
+            if (a.gate && a.gate_heads) inv *= 1.f / (1.f + __expf(-a.gate[(size_t)(row0 + qrow) * a.g_stride + head]));
+            bf16* o = a.out + (size_t)(row0 + qrow) * a.o_stride + head * DV;
+            const float* gt = (a.gate && !a.gate_heads) ? a.gate + (size_t)(row0 + qrow) * a.g_stride + head * DV : nullptr;
 #pragma unroll
-            for (int i = 0; i < D / 8; ++i) {
+            for (int i = 0; i < DV / 8; ++i) {
                 uint32_t hi, lo;
                 float o0 = o_acc[i][2 * r] * inv, o1 = o_acc[i][2 * r + 1] * inv;
                 if (gt) {        // sigmoid output gate, in f32
@@ -528,27 +552,33 @@ flash_prefill_kernel(FlashArgs a) {
     }
 }
 
-template <int D, bool CAUSAL, bool PAGED, bool SPLIT>
+template <int D, int DV, bool CAUSAL, bool PAGED, bool SPLIT>
 static int flash_launch_t(cudaStream_t st, const FlashArgs& a) {
-    constexpr int P = SPLIT ? 2 : 1, GROUPS = 2, BN = (SPLIT || D > 128) ? 32 : 64, STG = (SPLIT && D > 128) ? 1 : 2;
-    constexpr int SMEM = (P * 64 * (D + 8) + GROUPS * STG * 2 * P * BN * (D + 8)) * 2;
-    static_assert(STG * 2 * P * BN * (D + 8) * 2 >= 128 * (D / 2 + 4) * 4, "the merge buffer lives in group 1's ring");
+    constexpr int P = SPLIT ? 2 : 1, GROUPS = 2, DM = D > DV ? D : DV, BN = (SPLIT || DM > 128) ? 32 : 64, STG = (SPLIT && DM > 128) ? 1 : 2;
+    constexpr int SMEM = (P * 64 * (D + 8) + GROUPS * STG * P * BN * (D + DV + 16)) * 2;
+    static_assert(STG * P * BN * (D + DV + 16) * 2 >= 128 * (DV / 2 + 4) * 4, "the merge buffer lives in group 1's ring");
     static_assert(SMEM <= 227 * 1024, "flash tile does not fit");
     static SmemOptIn seen;
-    if (const int e = ensure_dyn_smem(flash_prefill_kernel<D, CAUSAL, PAGED, SPLIT>, (size_t)SMEM, seen)) return e;
+    if (const int e = ensure_dyn_smem(flash_prefill_kernel<D, DV, CAUSAL, PAGED, SPLIT>, (size_t)SMEM, seen)) return e;
     const int max_len = a.seq_len ? a.max_len : a.S;
     dim3 grid((max_len + 63) / 64, a.nh, a.seq_len ? a.nseq : 1);
-    return launch_k(flash_prefill_kernel<D, CAUSAL, PAGED, SPLIT>, grid, dim3(256), SMEM, st, prefill_pdl(), a);
+    return launch_k(flash_prefill_kernel<D, DV, CAUSAL, PAGED, SPLIT>, grid, dim3(256), SMEM, st, prefill_pdl(), a);
 }
 
-int flash_prefill_launch(cudaStream_t st, int D, bool causal, bool paged, const FlashArgs& a) {
+int flash_prefill_launch(cudaStream_t st, int D, bool causal, bool paged, const FlashArgs& a, int DV) {
     const bool split = a.q_lo_off != 0;
     if (split && (a.kv_lo_off == 0 || a.out_lo_off == 0)) return -1000;
-    if (D == 64 && causal && paged) return split ? flash_launch_t<64, true, true, true>(st, a) : flash_launch_t<64, true, true, false>(st, a);
-    if (D == 128 && causal && paged) return split ? flash_launch_t<128, true, true, true>(st, a) : flash_launch_t<128, true, true, false>(st, a);
-    if (D == 256 && causal && paged) return split ? flash_launch_t<256, true, true, true>(st, a) : flash_launch_t<256, true, true, false>(st, a);
-    if (D == 64 && !causal && !paged) return split ? flash_launch_t<64, false, false, true>(st, a) : flash_launch_t<64, false, false, false>(st, a);
-    if (D == 128 && !causal && !paged) return split ? flash_launch_t<128, false, false, true>(st, a) : flash_launch_t<128, false, false, false>(st, a);
+    if (DV != 0 && DV != D) {
+        if (!causal || !paged) return -1000;
+        if (D == 64 && DV == 128) return split ? flash_launch_t<64, 128, true, true, true>(st, a) : flash_launch_t<64, 128, true, true, false>(st, a);
+        if (D == 128 && DV == 64) return split ? flash_launch_t<128, 64, true, true, true>(st, a) : flash_launch_t<128, 64, true, true, false>(st, a);
+        return -1000;
+    }
+    if (D == 64 && causal && paged) return split ? flash_launch_t<64, 64, true, true, true>(st, a) : flash_launch_t<64, 64, true, true, false>(st, a);
+    if (D == 128 && causal && paged) return split ? flash_launch_t<128, 128, true, true, true>(st, a) : flash_launch_t<128, 128, true, true, false>(st, a);
+    if (D == 256 && causal && paged) return split ? flash_launch_t<256, 256, true, true, true>(st, a) : flash_launch_t<256, 256, true, true, false>(st, a);
+    if (D == 64 && !causal && !paged) return split ? flash_launch_t<64, 64, false, false, true>(st, a) : flash_launch_t<64, 64, false, false, false>(st, a);
+    if (D == 128 && !causal && !paged) return split ? flash_launch_t<128, 128, false, false, true>(st, a) : flash_launch_t<128, 128, false, false, false>(st, a);
     return -1000;
 }
 

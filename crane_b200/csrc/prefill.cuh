@@ -65,6 +65,9 @@ struct FlashArgs {
     float softcap = 0.f;
     const float* dist_r1 = nullptr; const float* dist_r2 = nullptr;
     const float* dist_table = nullptr; int dist_rows = 0;
+    int keep_first = 0;                 // window > 0: the first keep_first keys of the sequence stay visible behind the window
+    int gate_heads = 0;                 // 1: gate holds one number per head ([rows, g_stride], head h at h)
+    float out_mult = 1.f;               // factor on every output
 };
 
 // quantised KV pages <-> the bf16 (hi + lo) scratch the prefill kernels read and write (see prefill.cu)
@@ -84,7 +87,9 @@ int embed_rows_launch(cudaStream_t st, const uint32_t* ids, int S, const bf16* e
 int rmsnorm_rows_launch(cudaStream_t st, const float* x, int S, int H, const float* w, float eps, bf16* out, long long lo_off = 0);
 int layernorm_rows_launch(cudaStream_t st, const float* x, int rows, int W, const float* w, const float* b, float eps, bf16* out, long long lo_off = 0);
 int rope_append_launch(cudaStream_t st, int D, const RopeAppendArgs& a);
-int flash_prefill_launch(cudaStream_t st, int D, bool causal, bool paged, const FlashArgs& a);
+// D: key width; DV: value width (0: equal).  Widths that differ: paged causal launches with (64, 128) or (128, 64); flash_widths_fit tells.
+int flash_prefill_launch(cudaStream_t st, int D, bool causal, bool paged, const FlashArgs& a, int DV = 0);
+inline bool flash_widths_fit(int D, int DV) { return (D == DV && (D == 64 || D == 128 || D == 256)) || (D == 64 && DV == 128) || (D == 128 && DV == 64); }
 int gate_mul_launch(cudaStream_t st, bf16* attn, const float* qkv, int S, int nh, int D, int q_stride, int row_width, long long lo_off = 0);
 int set_rows_launch(cudaStream_t st, float* x, int H, const int* rows, int n, const float* src, bool add);
 int cast_f32_bf16_launch(cudaStream_t st, const float* src, bf16* dst, size_t n, long long lo_off = 0);

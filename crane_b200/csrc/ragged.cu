@@ -36,7 +36,7 @@ __global__ void embed_sinpos_rows_kernel(const int* __restrict__ ids, const int*
 // Block per row.  One input: x += rms(y1 + b1) * norm_w.  Two inputs: v = (rms(y1 + b1) * w1 + rms(y2) * w2) / 2, x += rms(v) * norm_w.
 __global__ void __launch_bounds__(256) post_norm_add_kernel(const float* __restrict__ y1, int ld1, const float* __restrict__ b1, const float* __restrict__ w1,
                                                             const float* __restrict__ y2, int ld2, const float* __restrict__ w2,
-                                                            const float* __restrict__ norm_w, float eps, float* __restrict__ x, int ldx, int W, ActOut planes) {
+                                                            const float* __restrict__ norm_w, float eps, float* __restrict__ x, int ldx, int W, ActOut planes, DytNorm dyt) {
     __shared__ float red[3][8];
     const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const float* a = y1 + (size_t)r * ld1;
@@ -58,11 +58,12 @@ __global__ void __launch_bounds__(256) post_norm_add_kernel(const float* __restr
         if (b) sb = fmaf(b[c], b[c], sb);
     }
     const float ia = 1.f / sqrtf(total(sa, 0) / (float)W + eps);
+    const float al = dyt.w ? *dyt.alpha : 0.f;
     if (!b) {
         for (int c = threadIdx.x; c < W; c += 256) {
             const float nx = xr[c] + (a[c] + (b1 ? b1[c] : 0.f)) * ia * norm_w[c];
             xr[c] = nx;
-            store_act(planes, r, c, nx);
+            store_act(planes, r, c, dyt.w ? tanhf(al * nx) * dyt.w[c] + dyt.b[c] : nx);
         }
         return;
     }
@@ -77,7 +78,7 @@ __global__ void __launch_bounds__(256) post_norm_add_kernel(const float* __restr
         const float v = 0.5f * ((a[c] + (b1 ? b1[c] : 0.f)) * ia * (w1 ? w1[c] : 1.f) + b[c] * ib * (w2 ? w2[c] : 1.f));
         const float nx = xr[c] + v * iv * norm_w[c];
         xr[c] = nx;
-        store_act(planes, r, c, nx);
+        store_act(planes, r, c, dyt.w ? tanhf(al * nx) * dyt.w[c] + dyt.b[c] : nx);
     }
 }
 
@@ -133,7 +134,7 @@ __global__ void gather_rows_kernel(const float* __restrict__ src, int lds, const
 template <int MODE>
 __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict__ A, int lda, const bf16* __restrict__ Wt, int ldw, int M, int N,
                                                          int K, float* __restrict__ C, int ldc, const float* __restrict__ col_scale,
-                                                         const float* __restrict__ gate, int ldg, const float* __restrict__ gate_bias) {
+                                                         const float* __restrict__ gate, int ldg, const float* __restrict__ gate_bias, const float* __restrict__ bias) {
     __shared__ float sa[16][64 + 4], sw[16][64 + 4];
     const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64, tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
     float acc[4][4] = {};
@@ -169,6 +170,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict
             if (m < M && n < N) {
                 float* p = C + (size_t)m * ldc + n;
                 float v = acc[i][j];
+                if (MODE == LIN_RESID && bias) v += bias[n];
                 if (MODE == LIN_RESID && col_scale) v *= col_scale[n];
                 if (MODE == LIN_RESID && gate) v *= 1.f / (1.f + expf(-(gate[(size_t)m * ldg + n] + (gate_bias ? gate_bias[n] : 0.f))));
                 *p = (MODE == LIN_RESID) ? *p + v : v;
@@ -194,7 +196,7 @@ __global__ void attn_prep_kernel(RaggedBatch rb, AttnPrepArgs a) {
         for (int i = threadIdx.x; i < nrot; i += blockDim.x) {
             double sn, cs;
             sincos((double)pos * a.rot_freq[i], &sn, &cs);
-            rot_cs[i] = (float)cs; rot_cs[nrot + i] = (float)sn;
+            rot_cs[i] = (float)cs * a.rot_mag; rot_cs[nrot + i] = (float)sn * a.rot_mag;
         }
         __syncthreads();
     }
@@ -219,7 +221,46 @@ __global__ void attn_prep_kernel(RaggedBatch rb, AttnPrepArgs a) {
     float temp = 1.f;
     if (a.temp_every > 0) temp = 1.f + a.temp_coef * logf((float)((pos + 1) / a.temp_every) + 1.f);
     const int page = a.has_kv ? a.block_table[(size_t)slot * a.max_pages + pos / KV_PAGE] : 0;
+    // value of a projected column: as it is (+ bias), or behind the short convolution over time (a channel belongs to one lane, which
+    // also moves the channel's window on in a step of single rows)
+    const int taps = a.conv_w ? a.conv_taps : 0, conv_ch = (a.H + a.G) * a.d + a.G * a.dv, row_in = r - rb.ent_row0[e];
+    float* win = taps > 1 ? a.conv_state + (size_t)slot * (taps - 1) * conv_ch : nullptr;
+    auto projected = [&](int c) -> float {
+        const float own = row[c];
+        if (!taps) return own + (a.bias ? a.bias[c] : 0.f);
+        const float* w = a.conv_w + (size_t)c * taps;
+        float acc = 0.f;
+        for (int k = 0; k < taps - 1; ++k) {
+            const int back = taps - 1 - k;                // this tap reads the projection `back` tokens ago
+            acc = fmaf(w[k], row_in >= back ? row[c - (ptrdiff_t)back * a.ld] : win[(size_t)(row_in + k) * conv_ch + c], acc);
+        }
+        if (a.single_rows && taps > 1) {
+            for (int k = 1; k < taps - 1; ++k) win[(size_t)(k - 1) * conv_ch + c] = win[(size_t)k * conv_ch + c];
+            win[(size_t)(taps - 2) * conv_ch + c] = own;
+        }
+        return fmaf(w[taps - 1], own, acc);
+    };
     for (int hh = warp; hh < nheads; hh += nw) {
+        if (taps || a.rot_halves) {      // convolved projections and / or the halves-paired rotation: no norm, no temperature
+            const bool isv = hh >= a.H + a.G, isq = hh < a.H;
+            const int width = isv ? a.dv : a.d, half = isv ? 0 : nrot, c0 = isv ? (a.H + a.G) * a.d + (hh - a.H - a.G) * a.dv : hh * a.d;
+            KT* dst = nullptr;
+            if (!isq) {
+                const int g = isv ? hh - a.H - a.G : hh - a.H;
+                dst = (KT*)(isv ? a.v_pool : a.k_pool) + (((size_t)page * a.G + g) * KV_PAGE + (pos % KV_PAGE)) * width;
+            }
+            auto put = [&](int c, float v) {
+                if (isq) store_act(a.q_out, r, c0 + c, v);
+                else kv_store<KT>(dst + c, v, a.kv_lo_off);
+            };
+            for (int i = lane; i < half; i += 32) {
+                const float u = projected(c0 + i), v = projected(c0 + i + half), cs = rot_cs[i], sn = rot_cs[half + i];
+                put(i, u * cs - v * sn);
+                put(i + half, v * cs + u * sn);
+            }
+            for (int c = 2 * half + lane; c < width; c += 32) put(c, projected(c0 + c));
+            continue;
+        }
         if (hh < a.H + nk) {             // q or k head: RMS norm over d (or the row's whole-projection statistic)
             const bool isq = hh < a.H;
             const float* src = row + (size_t)hh * a.d;
@@ -298,6 +339,11 @@ template <> __device__ __forceinline__ void kv_load8<bf16>(const bf16* p, long l
         v[4] += bf16lo(l.z); v[5] += bf16hi(l.z); v[6] += bf16lo(l.w); v[7] += bf16hi(l.w);
     }
 }
+// factor on an attention output: the sigmoid gate (one per output or one per head) and the constant
+__device__ __forceinline__ float attn_out_factor(const SinkAttnArgs& a, int r, int h, int col) {
+    if (!a.gate) return a.out_mult;
+    return a.out_mult / (1.f + __expf(-a.gate[(size_t)r * a.ldg + (a.gate_heads ? h : h * a.dv + col)]));
+}
 template <typename KT, int REP, bool STAGE>
 __global__ void __launch_bounds__(ATT_WARPS * 32) sink_attention_kernel(RaggedBatch rb, SinkAttnArgs a) {
     constexpr bool stage = STAGE;
@@ -316,8 +362,10 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) sink_attention_kernel(RaggedBa
     const int nkeys = pos + 1;
     const int key0 = (a.window > 0 && nkeys > a.window) ? nkeys - a.window : 0;      // first key the row sees
     const int t0 = key0 / 32;                            // (its tile holds at least that key: no tile is hidden entirely)
-    const int ntiles = (nkeys + 31) / 32, per = (ntiles - t0 + a.nsplit - 1) / a.nsplit;
-    const int t_lo = t0 + sp * per, t_hi = min(ntiles, t_lo + per);
+    const int keep = key0 > 0 ? a.keep_first : 0;        // tokens visible behind the window
+    const int nkt = min((keep + 31) / 32, t0);           // their tiles come first, those that the window does not reach
+    const int ntiles = (nkeys + 31) / 32, per = (nkt + ntiles - t0 + a.nsplit - 1) / a.nsplit;
+    const int t_lo = sp * per, t_hi = min(nkt + ntiles - t0, t_lo + per);
     float m[REP], l[REP], acc[REP][ATT_MAXC];
 #pragma unroll
     for (int q = 0; q < REP; ++q) {
@@ -341,7 +389,8 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) sink_attention_kernel(RaggedBa
         vst = one_copy ? kst : kst + (size_t)32 * planes * ks_e;
     }
     const long long klo = !stage ? a.kv_lo_off : planes == 2 ? (long long)32 * ks_e : 0, vlo = !stage ? a.kv_lo_off : planes == 2 ? (long long)32 * vs_e : 0;
-    for (int t = t_lo + warp; t < t_hi; t += ATT_WARPS) {
+    for (int ti = t_lo + warp; ti < t_hi; ti += ATT_WARPS) {
+        const int t = ti < nkt ? ti : t0 + ti - nkt;
         const int j = t * 32 + lane;
         const int pg = bt[(t * 32) / KV_PAGE];           // a 32-key tile never straddles a 64-token page
         const size_t base = ((size_t)pg * a.G + g) * KV_PAGE + ((t * 32) % KV_PAGE);
@@ -369,7 +418,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) sink_attention_kernel(RaggedBa
         float sc[REP];
 #pragma unroll
         for (int q = 0; q < REP; ++q) sc[q] = 0.f;
-        const bool seen = j < nkeys && j >= key0;
+        const bool seen = j < nkeys && (j >= key0 || j < keep);
         if (seen) {
             const KT* kr = stage ? kst + (size_t)lane * ks_e : (const KT*)a.k_pool + (base + lane) * d;
             if (kvec) {
@@ -487,7 +536,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) sink_attention_kernel(RaggedBa
         for (int col = threadIdx.x; col < dv; col += blockDim.x) {
             float o = 0.f;
             for (int w = 0; w < ATT_WARPS; ++w) o += wa[((size_t)w * REP + q) * dv + col] * wsc[w];
-            if (last) store_act(a.out, r, h * dv + col, o / Lsum * (a.gate ? 1.f / (1.f + __expf(-a.gate[(size_t)r * a.ldg + h * dv + col])) : 1.f));
+            if (last) store_act(a.out, r, h * dv + col, o / Lsum * attn_out_factor(a, r, h, col));
             else a.part[(((size_t)r * a.H + h) * a.nsplit + sp) * (dv + 2) + 2 + col] = o;
         }
         if (!last && threadIdx.x == 0) {
@@ -519,7 +568,7 @@ __global__ void sink_attention_merge_kernel(SinkAttnArgs a) {
         float o = 0.f;
 #pragma unroll 4
         for (int sp = 0; sp < ns; ++sp) o = fmaf(pp[(size_t)sp * (dv + 2) + 2 + col], wgt[sp], o);
-        store_act(a.out, r, h * dv + col, o * invL * (a.gate ? 1.f / (1.f + __expf(-a.gate[(size_t)r * a.ldg + h * dv + col])) : 1.f));
+        store_act(a.out, r, h * dv + col, o * invL * attn_out_factor(a, r, h, col));
     }
 }
 
@@ -741,10 +790,10 @@ __global__ void clamped_glu_kernel(const float* __restrict__ gu, int ld, int str
     store_act(out, r, j, g / (1.f + __expf(-1.702f * g)) * (u + 1.f));
 }
 
-__global__ void silu_glu_kernel(const float* __restrict__ gu, int ld, int F, ActOut out, float limit) {
+__global__ void silu_glu_kernel(const float* __restrict__ gu, int ld, int F, ActOut out, float limit, const float* __restrict__ bias) {
     const int r = blockIdx.y, j = blockIdx.x * blockDim.x + threadIdx.x;
     if (j >= F) return;
-    store_act(out, r, j, glu_pair_f(gu[(size_t)r * ld + 2 * j], gu[(size_t)r * ld + 2 * j + 1], limit < 0.f ? limit : 0.f));
+    store_act(out, r, j, glu_pair_f(gu[(size_t)r * ld + 2 * j] + (bias ? bias[2 * j] : 0.f), gu[(size_t)r * ld + 2 * j + 1] + (bias ? bias[2 * j + 1] : 0.f), limit < 0.f ? limit : 0.f));
 }
 
 // Router logits of one row by one warp: NB experts at a time share the loads of the f32 row; a lane owns 8 neighbouring columns per
@@ -1094,9 +1143,9 @@ int embed_sinpos_rows_launch(cudaStream_t st, const int* ids, const int* row_pos
     return last_err();
 }
 int post_norm_add_launch(cudaStream_t st, const float* y1, int ld1, const float* b1, const float* w1, const float* y2, int ld2, const float* w2,
-                         const float* norm_w, float eps, float* x, int ldx, int T, int W, const ActOut& planes) {
-    if (!y1 || !norm_w || planes.f) return -1000;
-    post_norm_add_kernel<<<T, 256, 0, st>>>(y1, ld1, b1, w1, y2, ld2, w2, norm_w, eps, x, ldx, W, planes);
+                         const float* norm_w, float eps, float* x, int ldx, int T, int W, const ActOut& planes, const DytNorm& dyt) {
+    if (!y1 || !norm_w || (planes.f && !dyt.w)) return -1000;
+    post_norm_add_kernel<<<T, 256, 0, st>>>(y1, ld1, b1, w1, y2, ld2, w2, norm_w, eps, x, ldx, W, planes, dyt);
     return last_err();
 }
 int dyt_rows_launch(cudaStream_t st, const float* x, int ldx, const int* rows, int R, int W, const float* alpha, const float* w, const float* b,
@@ -1117,11 +1166,11 @@ int gather_rows_launch(cudaStream_t st, const float* src, int lds, const int* ro
     return last_err();
 }
 int linear_f32_launch(cudaStream_t st, const float* A, int lda, const bf16* W, int ldw, int M, int N, int K, int mode, float* C, int ldc,
-                      const float* col_scale, const float* gate, int ldg, const float* gate_bias) {
+                      const float* col_scale, const float* gate, int ldg, const float* gate_bias, const float* bias) {
     if (M <= 0 || N <= 0 || K <= 0) return -1000;
     const dim3 grid((N + 63) / 64, (M + 63) / 64);
-    if (mode == LIN_RESID) linear_f32_kernel<LIN_RESID><<<grid, 256, 0, st>>>(A, lda, W, ldw, M, N, K, C, ldc, col_scale, gate, ldg, gate_bias);
-    else linear_f32_kernel<LIN_STORE><<<grid, 256, 0, st>>>(A, lda, W, ldw, M, N, K, C, ldc, nullptr, nullptr, 0, nullptr);
+    if (mode == LIN_RESID) linear_f32_kernel<LIN_RESID><<<grid, 256, 0, st>>>(A, lda, W, ldw, M, N, K, C, ldc, col_scale, gate, ldg, gate_bias, bias);
+    else linear_f32_kernel<LIN_STORE><<<grid, 256, 0, st>>>(A, lda, W, ldw, M, N, K, C, ldc, nullptr, nullptr, 0, nullptr, nullptr);
     return last_err();
 }
 int rms_rows_launch(cudaStream_t st, const float* x, int ldx, const int* rows, int R, int W, float eps, const float* w1, const ActOut& out1,
@@ -1134,13 +1183,15 @@ int store_rows_launch(cudaStream_t st, const float* src, int lds, int T, int W, 
     store_rows_kernel<<<T, 128, 0, st>>>(src, lds, W, dst, col0);
     return last_err();
 }
-int silu_glu_launch(cudaStream_t st, const float* gu, int ld, int T, int F, const ActOut& out, float limit) {
-    silu_glu_kernel<<<dim3((F + 127) / 128, T), 128, 0, st>>>(gu, ld, F, out, limit);
+int silu_glu_launch(cudaStream_t st, const float* gu, int ld, int T, int F, const ActOut& out, float limit, const float* bias) {
+    silu_glu_kernel<<<dim3((F + 127) / 128, T), 128, 0, st>>>(gu, ld, F, out, limit, bias);
     return last_err();
 }
 int attn_prep_launch(cudaStream_t st, const RaggedBatch& rb, const AttnPrepArgs& a) {
     if (a.rot_dims < 0 || (a.rot_dims & 1) || a.rot_dims > a.d || a.rot_dims > 4096) return -1000;
     if (a.v_from_k && a.d != a.dv) return -1000;
+    if ((a.conv_w || a.rot_halves) && (!a.no_norm || !a.has_kv || a.v_from_k || a.v_unit || a.bias || a.q_head_scale)) return -1000;
+    if (a.conv_w && (a.conv_taps < 1 || (a.conv_taps > 1 && !a.conv_state))) return -1000;
     const size_t sm = (size_t)a.rot_dims * sizeof(float);
     if (a.kv_f32) attn_prep_kernel<float><<<rb.T, 256, sm, st>>>(rb, a);
     else attn_prep_kernel<bf16><<<rb.T, 256, sm, st>>>(rb, a);
@@ -1178,7 +1229,7 @@ static int sink_attention_launch_k(cudaStream_t st, const RaggedBatch& rb, const
     return sink_attention_launch_t<KT, 8>(st, rb, a);
 }
 int sink_attention_launch(cudaStream_t st, const RaggedBatch& rb, const SinkAttnArgs& a) {
-    if (a.dv > 32 * ATT_MAXC || a.H % a.G) return -1000;
+    if (a.dv > 32 * ATT_MAXC || a.H % a.G || a.keep_first < 0) return -1000;
     if (a.kv_shared && (a.k_pool != a.v_pool || a.d != a.dv)) return -1000;
     int e = a.kv_f32 ? sink_attention_launch_k<float>(st, rb, a) : sink_attention_launch_k<bf16>(st, rb, a);
     if (e || a.nsplit == 1) return e;

@@ -14,7 +14,8 @@
 //   whose sublayers read the stream itself and are normalised on their way back: a sinusoidal position vector on the embedding, the
 //   post-norm residual add (one or two normalised inputs), attention scores with a tanh cap, a logarithmic distance penalty or a
 //   distance table, projection biases, a whole-projection norm, unit-RMS values or values taken from the raw keys (ragged.cu), and,
-//   in ragged_scan.cu, the Mamba-1 selective scan and the mLSTM matrix memory.
+//   in ragged_scan.cu, the Mamba-1 selective scan and the mLSTM matrix memory.  In ragged_delta.cu: the gated delta rule with a decay per
+//   head or per key channel, and an embedding of the token that joins behind every layer.
 #pragma once
 
 #include "common.cuh"
@@ -46,9 +47,10 @@ int embed_sinpos_rows_launch(cudaStream_t st, const int* ids, const int* row_pos
 // Norm on a sublayer's way back into the stream.  One input: x[r] += rms(y1[r] + b1) * norm_w.  Two inputs (y2 != nullptr): each is
 // RMS-normed with its own weight first and half their sum takes y1's place: v = (rms(y1 + b1) * w1 + rms(y2) * w2) / 2.
 // b1, w1, w2 nullable.  Every mean of squares runs thread-strided, then over a fixed tree.  planes (optional): the new x also leaves as
-// bf16 operand planes, for the linear that reads the stream next.
+// bf16 operand planes, for the linear that reads the stream next -- or, with `dyt` (alpha, w, b of a Dynamic-Tanh norm), that norm of it.
+struct DytNorm { const float *alpha = nullptr, *w = nullptr, *b = nullptr; };
 int post_norm_add_launch(cudaStream_t st, const float* y1, int ld1, const float* b1, const float* w1, const float* y2, int ld2, const float* w2,
-                         const float* norm_w, float eps, float* x, int ldx, int T, int W, const ActOut& planes = ActOut{});
+                         const float* norm_w, float eps, float* x, int ldx, int T, int W, const ActOut& planes = ActOut{}, const DytNorm& dyt = DytNorm{});
 // out[r, c] = tanh(alpha * x[src(r), c]) * w[c] + b[c];  rows = gather list (nullptr: identity)
 int dyt_rows_launch(cudaStream_t st, const float* x, int ldx, const int* rows, int R, int W, const float* alpha, const float* w,
                     const float* b, const ActOut& out);
@@ -60,12 +62,13 @@ int rms_rows_launch(cudaStream_t st, const float* x, int ldx, const int* rows, i
 // dst[r, col0 + c] = src[r, c] for c < W, in every form dst carries (f32 rows, bf16 planes)
 int store_rows_launch(cudaStream_t st, const float* src, int lds, int T, int W, const ActOut& dst, int col0);
 // C[M, N] (+)= A[M, K] f32 x W[N, K]^T bf16, every product and sum in f32 (no tensor cores): the exact mode's linear, and the router's.
-// col_scale (LIN_RESID only, nullable): C[m, n] += col_scale[n] * acc;  gate (LIN_RESID only, nullable [M, ldg], gate_bias nullable [N]):
+// bias, col_scale (LIN_RESID only, nullable): C[m, n] += col_scale[n] * (acc + bias[n]);  gate (LIN_RESID only, nullable [M, ldg], gate_bias nullable [N]):
 // the added value is also multiplied by sigmoid(gate[m, n] + gate_bias[n])
 int linear_f32_launch(cudaStream_t st, const float* A, int lda, const bf16* W, int ldw, int M, int N, int K, int mode, float* C, int ldc,
-                      const float* col_scale = nullptr, const float* gate = nullptr, int ldg = 0, const float* gate_bias = nullptr);
-// out[r, j] = silu(gu[r, 2j]) * gu[r, 2j + 1]  (interleaved (gate, up) pairs);  limit < 0: gelu_tanh in place of silu
-int silu_glu_launch(cudaStream_t st, const float* gu, int ld, int T, int F, const ActOut& out, float limit = 0.f);
+                      const float* col_scale = nullptr, const float* gate = nullptr, int ldg = 0, const float* gate_bias = nullptr, const float* bias = nullptr);
+// out[r, j] = silu(gu[r, 2j]) * gu[r, 2j + 1]  (interleaved (gate, up) pairs);  limit < 0: gelu_tanh in place of silu;
+// bias (nullable [2 F], interleaved like gu) joins first
+int silu_glu_launch(cudaStream_t st, const float* gu, int ld, int T, int F, const ActOut& out, float limit = 0.f, const float* bias = nullptr);
 
 struct AttnPrepArgs {
     const float* qkv; int ld;         // [T, ld]: q heads | k heads | v heads (k / v absent when has_kv == 0)
@@ -88,6 +91,14 @@ struct AttnPrepArgs {
     int v_unit = 0;                   // 1: every value head is divided by its root mean square over dv (eps, no weight) before it is cached
     int v_from_k = 0;                 // 1: the row has no value columns; the cached value of a head is its key as projected (+ bias), before the norm (dv == d)
     const float* q_head_scale = nullptr;   // nullable [H]: head h's normalised query is multiplied by q_head_scale[h]
+    int rot_halves = 0;               // 1: dimension i turns together with dimension i + rot_dims / 2 (instead of pairs (2i, 2i + 1))
+    float rot_mag = 1.f;              // factor on the rotation's cosines and sines
+    // a short causal convolution over time on every projected channel (q | k | v columns), ahead of everything else:
+    // u_t = sum_j conv_w[c, j] * p_(t - taps + 1 + j), p the projections; inputs ahead of the entry come from the carried window
+    const float* conv_w = nullptr;    // [(H + G) * d + G * dv, taps]
+    int conv_taps = 0;
+    float* conv_state = nullptr;      // [slots, taps - 1, channels]; moved on here when every entry brings one row, else by causal_conv_window_launch
+    int single_rows = 0;
 };
 int attn_prep_launch(cudaStream_t st, const RaggedBatch& rb, const AttnPrepArgs& a);
 
@@ -108,6 +119,9 @@ struct SinkAttnArgs {
     float softcap = 0.f;
     const float* dist_r1 = nullptr; const float* dist_r2 = nullptr;
     const float* dist_table = nullptr; int dist_rows = 0;
+    int keep_first = 0;                      // window > 0: the first keep_first tokens of the sequence stay visible behind the window
+    int gate_heads = 0;                      // 1: gate is [T, ldg] with one number per head: out[r, h * dv + c] *= sigmoid(gate[r, h])
+    float out_mult = 1.f;                    // factor on every output
 };
 int sink_attention_launch(cudaStream_t st, const RaggedBatch& rb, const SinkAttnArgs& a);
 
@@ -194,6 +208,8 @@ struct CausalConvArgs {
 };
 int causal_conv_launch(cudaStream_t st, const RaggedBatch& rb, const CausalConvArgs& a);
 int causal_conv_launch_count(const CausalConvArgs& a);
+// the window alone: the sequences' windows become their last taps - 1 inputs (in, ld, C, taps, state of `a`)
+int causal_conv_window_launch(cudaStream_t st, const RaggedBatch& rb, const CausalConvArgs& a);
 
 // Every entry one row: out_h = rms_in_groups(x) * norm_w, out_u = out_h + conv(out_h) over the carried window, window moved on -- one launch,
 // for the sizes norm_conv_step_fits() accepts (the others take rms_rows + causal_conv)
@@ -295,6 +311,41 @@ int mlstm_mixer_launch(cudaStream_t st, const RaggedBatch& rb, const MlstmArgs& 
 int mlstm_launch_count(bool has_seg_scratch, int max_len);
 size_t mlstm_seg_floats(int entries, int H, int d, int dv);
 size_t mlstm_seg_decay_offset(int entries, int H, int d, int dv);
+
+// ---- the gated delta rule (ragged_delta.cu) ---------------------------------------------------------------------------------------------
+// proj [T, ld] holds, from column col0 on, q | k | v (Hk*d, Hk*d, H*dv columns); the step sizes' pre-activations (H columns) start at b_col.
+// Every channel of q, k, v passes a causal convolution over time (carried window) and SiLU; q and k become unit vectors per head,
+// x / sqrt(sum(x^2) + 1e-6), q also times q_scale; head h reads q / k head h / (H / Hk).  With beta = sigmoid(b), all in f32:
+//   S <- decay S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+// decay = exp(-rate_h softplus(z + dt_bias)), per head (z [T, H], dt_bias [H]) or, with per_channel, per head and row of S (z [T, H*d],
+// dt_bias [H*d]).  out[r, out_col + h*dv + c] = out_mult * o / sqrt(mean_dv(o^2) + eps) * norm_w[c] * gate(g), gate = sigmoid or silu.
+// The state [slots, H, d, dv] is f32 and carried in place, the windows [slots, taps - 1, 2*Hk*d + H*dv] likewise.
+struct DeltaArgs {
+    const float* proj; int ld; int col0, b_col;
+    int Hk, H, d, dv, taps;
+    const float* conv_w;              // [2*Hk*d + H*dv, taps]
+    float* conv_state;
+    int single_rows;                  // every entry brings one row
+    float q_scale, eps, out_mult;
+    const float* z; int ldz; int per_channel;
+    const float* rate;                // [H] exp(A_log)
+    const float* dt_bias;
+    const float* g; int ldg; int gate_silu;
+    const float* norm_w;              // [dv]
+    float* state;
+    float *qn, *kn, *v, *beta, *qk, *y;         // scratch: [T, Hk*d] x 2, [T, H*dv], [T, H], [T, Hk], [T, H*dv]
+    float* dec; int lddec;            // scratch [T, lddec] for the decays, H*d or H columns (per channel: may be z itself)
+    ActOut out; int out_col;          // [T, .. out_col + H*dv]
+    int max_len = 0;                  // rows of the longest entry
+};
+int delta_mixer_launch(cudaStream_t st, const RaggedBatch& rb, const DeltaArgs& a);
+int delta_launch_count(const DeltaArgs& a);
+
+// A token's own embedding behind a layer: out[r, j] = gelu_tanh(z[r, j]) * table[ids[r], col0 + j], j < n (table [V, ldt] bf16)
+int token_gate_launch(cudaStream_t st, const float* z, int ldz, int T, int n, const int* ids, const bf16* table, int ldt, int col0, const ActOut& out);
+// ... with z = x w^T taken in the same launch, for a few rows: x [T, ldx] f32, w [n, ldw] bf16, K (multiple of 8) columns
+int token_gate_step_launch(cudaStream_t st, const float* x, int ldx, const bf16* w, int ldw, int K, int T, int n, const int* ids, const bf16* table, int ldt,
+                           int col0, const ActOut& out);
 
 // dst[r, c] = cap * tanh(src[r, c] / cap) for c < V (cap <= 0: a plain copy)
 int softcap_rows_launch(cudaStream_t st, const float* src, int lds, int R, int V, float cap, float* dst, int ldd);

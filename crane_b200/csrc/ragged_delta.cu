@@ -1,0 +1,394 @@
+// The gated delta rule on ragged batches (see ragged.cuh), and the embedding of the token that joins behind a layer.
+//   prep : per (q / k head | value head | gates): convolution over time with the carried window, SiLU, unit norms, q . k, the decays
+//          and step sizes -- f32 throughout, one warp per head and tile of rows, the tap window in registers;
+//   scan : the recurrence token by token, a thread keeps its share of the state in registers for the whole portion, the inputs of
+//          DR_CH tokens at a time staged in shared memory (cp.async, double-buffered);
+//   out  : norm over the value width, gate.
+// A row's result depends on its own sequence only: the split of the state over lanes and the order of the lane sums are launch
+// constants.
+#include "ragged.cuh"
+#include "ragged_dev.cuh"
+
+#include <algorithm>
+
+namespace cb {
+
+namespace {
+
+inline int last_err() { return (int)cudaGetLastError(); }
+
+__device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+
+// ---------------------------------------------------------------------------------------------------------------- prep
+// Walks rows r0 .. r1 - 1 of NC * 32 channels starting at column c0 (lane owns c0 + lane + 32 i, i < NC, below c0 + width): emit(r, y) gets
+// the convolved values of row r.  TAPS > 0: the tap window lives in registers; TAPS == 0: any number of taps, read back from memory.
+template <int NC, int TAPS>
+struct ConvWalk {
+    float w[NC][TAPS > 0 ? TAPS : 1], h[NC][TAPS > 1 ? TAPS - 1 : 1];
+    int c0, width, lane, C;
+    __device__ __forceinline__ void init(const DeltaArgs& a, int c0_, int width_, int lane_) {
+        c0 = c0_; width = width_; lane = lane_; C = 2 * a.Hk * a.d + a.H * a.dv;
+        if constexpr (TAPS > 0) {
+#pragma unroll
+            for (int i = 0; i < NC; ++i) {
+                const int c = lane + 32 * i;
+#pragma unroll
+                for (int k = 0; k < TAPS; ++k) w[i][k] = c < width ? a.conv_w[(size_t)(c0 + c) * TAPS + k] : 0.f;
+            }
+        }
+    }
+    __device__ __forceinline__ float before(const DeltaArgs& a, int slot, int in_entry, int r, int c, int k) const {      // what tap k of row r reads
+        const int back = a.taps - 1 - k;
+        return in_entry >= back ? a.proj[(size_t)(r - back) * a.ld + a.col0 + c0 + c] : a.conv_state[((size_t)slot * (a.taps - 1) + in_entry + k) * C + c0 + c];
+    }
+    __device__ __forceinline__ void refill(const DeltaArgs& a, int slot, int in_entry, int r) {
+        if constexpr (TAPS > 1) {
+#pragma unroll
+            for (int i = 0; i < NC; ++i) {
+                const int c = lane + 32 * i;
+#pragma unroll
+                for (int k = 0; k < TAPS - 1; ++k) h[i][k] = c < width ? before(a, slot, in_entry, r, c, k) : 0.f;
+            }
+        }
+    }
+    // y[i] of row r from its own inputs x[i]; with `move` the carried window of the row's sequence moves on
+    __device__ __forceinline__ void step(const DeltaArgs& a, int slot, int in_entry, int r, const float* x, float* y, bool move) {
+#pragma unroll
+        for (int i = 0; i < NC; ++i) {
+            const int c = lane + 32 * i;
+            float acc = 0.f;
+            if constexpr (TAPS > 0) {
+#pragma unroll
+                for (int k = 0; k < TAPS - 1; ++k) acc = fmaf(w[i][k], h[i][k], acc);
+                acc = fmaf(w[i][TAPS - 1], x[i], acc);
+                if (TAPS > 1) {
+#pragma unroll
+                    for (int k = 0; k < TAPS - 2; ++k) h[i][k] = h[i][k + 1];
+                    h[i][TAPS - 2] = x[i];
+                    if (move && c < width) {
+#pragma unroll
+                        for (int k = 0; k < TAPS - 1; ++k) a.conv_state[((size_t)slot * (TAPS - 1) + k) * C + c0 + c] = h[i][k];
+                    }
+                }
+            } else if (c < width) {
+                for (int k = 0; k < a.taps - 1; ++k) acc = fmaf(a.conv_w[(size_t)(c0 + c) * a.taps + k], before(a, slot, in_entry, r, c, k), acc);
+                acc = fmaf(a.conv_w[(size_t)(c0 + c) * a.taps + a.taps - 1], x[i], acc);
+                if (move) {
+                    float* win = a.conv_state + (size_t)slot * (a.taps - 1) * C + c0 + c;
+                    for (int k = 1; k < a.taps - 1; ++k) win[(size_t)(k - 1) * C] = win[(size_t)k * C];
+                    win[(size_t)(a.taps - 2) * C] = x[i];
+                }
+            }
+            y[i] = acc;
+        }
+    }
+};
+
+constexpr int DP_ROWS = 16;      // rows a warp walks
+template <int NC, int TAPS>
+__global__ void __launch_bounds__(128) delta_prep_kernel(RaggedBatch rb, DeltaArgs a, int tile) {
+    const int lane = threadIdx.x & 31, unit = blockIdx.y * 4 + (threadIdx.x >> 5), r0 = blockIdx.x * tile, r1 = min(rb.T, r0 + tile);
+    const int Hk = a.Hk, H = a.H, d = a.d, dv = a.dv, n_dec = a.per_channel ? H : 0;
+    if (unit >= Hk + H + n_dec + 1) return;
+    if (unit < Hk) {                                          // a q / k head: convolution, SiLU, unit vectors, their product
+        ConvWalk<NC, TAPS> q, k;
+        q.init(a, unit * d, d, lane);
+        k.init(a, (Hk + unit) * d, d, lane);
+        for (int rb0 = r0; rb0 < r1; rb0 += 4) {              // four rows requested before the first is used
+            float xq[4][NC], xk[4][NC];
+#pragma unroll
+            for (int u = 0; u < 4; ++u)
+#pragma unroll
+                for (int i = 0; i < NC; ++i) {
+                    const bool ok = rb0 + u < r1 && lane + 32 * i < d;
+                    const float* p = a.proj + (size_t)(rb0 + u) * a.ld + a.col0 + unit * d + lane + 32 * i;
+                    xq[u][i] = ok ? p[0] : 0.f; xk[u][i] = ok ? p[Hk * d] : 0.f;
+                }
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                const int r = rb0 + u;
+                if (r >= r1) break;
+                const int e = rb.row_entry[r], in_entry = r - rb.ent_row0[e], slot = rb.ent_slot[e];
+                if (r == r0 || in_entry == 0) { q.refill(a, slot, in_entry, r); k.refill(a, slot, in_entry, r); }
+                float yq[NC], yk[NC], sq = 0.f, sk = 0.f, sqk = 0.f;
+                q.step(a, slot, in_entry, r, xq[u], yq, a.single_rows != 0 && a.taps > 1);
+                k.step(a, slot, in_entry, r, xk[u], yk, a.single_rows != 0 && a.taps > 1);
+#pragma unroll
+                for (int i = 0; i < NC; ++i) {
+                    yq[i] = silu_f(yq[i]); yk[i] = silu_f(yk[i]);
+                    sq = fmaf(yq[i], yq[i], sq); sk = fmaf(yk[i], yk[i], sk); sqk = fmaf(yq[i], yk[i], sqk);
+                }
+                sq = warp_sum(sq); sk = warp_sum(sk); sqk = warp_sum(sqk);
+                const float iq = a.q_scale / sqrtf(sq + 1e-6f), ik = 1.f / sqrtf(sk + 1e-6f);
+#pragma unroll
+                for (int i = 0; i < NC; ++i)
+                    if (lane + 32 * i < d) {
+                        const size_t o = ((size_t)r * Hk + unit) * d + lane + 32 * i;
+                        a.qn[o] = yq[i] * iq; a.kn[o] = yk[i] * ik;
+                    }
+                if (lane == 0) a.qk[(size_t)r * Hk + unit] = sqk * iq * ik;
+            }
+        }
+    } else if (unit < Hk + H) {                               // a value head
+        const int h = unit - Hk;
+        for (int cb = 0; cb < dv; cb += 32 * NC) {
+            ConvWalk<NC, TAPS> v;
+            v.init(a, 2 * Hk * d + h * dv + cb, min(32 * NC, dv - cb), lane);
+            for (int rb0 = r0; rb0 < r1; rb0 += 4) {
+                float x[4][NC];
+#pragma unroll
+                for (int u = 0; u < 4; ++u)
+#pragma unroll
+                    for (int i = 0; i < NC; ++i)
+                        x[u][i] = (rb0 + u < r1 && lane + 32 * i < v.width) ? a.proj[(size_t)(rb0 + u) * a.ld + a.col0 + v.c0 + lane + 32 * i] : 0.f;
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    const int r = rb0 + u;
+                    if (r >= r1) break;
+                    const int e = rb.row_entry[r], in_entry = r - rb.ent_row0[e], slot = rb.ent_slot[e];
+                    if (r == r0 || in_entry == 0) v.refill(a, slot, in_entry, r);
+                    float y[NC];
+                    v.step(a, slot, in_entry, r, x[u], y, a.single_rows != 0 && a.taps > 1);
+#pragma unroll
+                    for (int i = 0; i < NC; ++i) if (lane + 32 * i < v.width) a.v[((size_t)r * H + h) * dv + cb + lane + 32 * i] = silu_f(y[i]);
+                }
+            }
+        }
+    } else if (unit < Hk + H + n_dec) {                       // the decays of a head's key channels
+        const int h = unit - Hk - H;
+        const float rate = a.rate[h];
+        for (int c = lane; c < d; c += 32) {
+            const float b = a.dt_bias[h * d + c];
+#pragma unroll 4
+            for (int r = r0; r < r1; ++r) a.dec[(size_t)r * a.lddec + h * d + c] = expf(-rate * softplus_f(a.z[(size_t)r * a.ldz + h * d + c] + b));
+        }
+    } else {                                                  // step sizes (and the decays of whole heads)
+        for (int i = lane; i < (r1 - r0) * H; i += 32) {
+            const int r = r0 + i / H, h = i % H;
+            a.beta[(size_t)r * H + h] = sigmoid_f(a.proj[(size_t)r * a.ld + a.b_col + h]);
+            if (!a.per_channel) a.dec[(size_t)r * a.lddec + h] = expf(-a.rate[h] * softplus_f(a.z[(size_t)r * a.ldz + h] + a.dt_bias[h]));
+        }
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------------------- scan
+// Block = (entry, head, DR_COLS value columns); thread (pl, ns) owns rows ns * R .. ns * R + R - 1 of column p0 + pl of S in registers.
+// A token's two products with the decayed state -- S^T k for the correction, S^T q for the output -- are reduced over the eight lanes of
+// a column together; the output then is S^T q + (q . k) u, which is the read-out after the write.  Tokens go in groups of four whose
+// operands are read ahead of the first reduction; a group's tokens past the end have decay 1 and step size 0.
+constexpr int DR_NS = 8, DR_COLS = 16, DR_CH = 16;
+// a staged vector is cut into eight runs of R, from R = 4 on each followed by 4 pad floats: spreads the runs of a warp over all banks
+__host__ __device__ inline int dr_idx(int n, int R) { return R >= 4 ? n + 4 * (n / R) : n; }
+__host__ __device__ inline int dr_pad(int R) { return R >= 4 ? DR_NS * (R + 4) : DR_NS * R; }
+template <int R>
+__device__ __forceinline__ void load_run(const float* p, float* o) {
+    if constexpr ((R & 3) == 0) {
+#pragma unroll
+        for (int i = 0; i < R / 4; ++i) { const float4 t = reinterpret_cast<const float4*>(p)[i]; o[4 * i] = t.x; o[4 * i + 1] = t.y; o[4 * i + 2] = t.z; o[4 * i + 3] = t.w; }
+    } else {
+#pragma unroll
+        for (int i = 0; i < R; ++i) o[i] = p[i];
+    }
+}
+template <int R, bool PC>
+__global__ void __launch_bounds__(DR_COLS * DR_NS) delta_scan_kernel(RaggedBatch rb, DeltaArgs a) {
+    extern __shared__ __align__(16) float sm[];
+    constexpr int NV = PC ? 3 : 2;                            // staged vectors per token: q | k (| decay)
+    const int e = blockIdx.x, h = blockIdx.y, p0 = blockIdx.z * DR_COLS, ns = threadIdx.x & (DR_NS - 1), pl = threadIdx.x / DR_NS, p = p0 + pl;
+    const int d = a.d, dv = a.dv, H = a.H, Hk = a.Hk, hk = h / (H / Hk), DPD = dr_pad(R), PT = NV * DPD + DR_COLS + 4;
+    const bool live = p < dv;
+    const int len = rb.ent_len[e], slot = rb.ent_slot[e], r0 = rb.ent_row0[e], ncol = min(DR_COLS, dv - p0), n0 = ns * R;
+    float* stage[2] = {sm, sm + DR_CH * PT};
+    float* sy = sm + 2 * DR_CH * PT;                          // [CH][COLS]
+    for (int i = threadIdx.x; i < 2 * DR_CH * PT; i += blockDim.x) sm[i] = 0.f;       // rows past d, columns past dv stay zero
+    float* S = a.state + ((size_t)slot * H + h) * d * dv + (live ? p : 0);
+    float s[R];
+#pragma unroll
+    for (int i = 0; i < R; ++i) s[i] = (live && n0 + i < d) ? S[(size_t)(n0 + i) * dv] : 0.f;
+    __syncthreads();
+    const bool wide = ((d | dv | (PC ? a.lddec : 0)) & 3) == 0 && R >= 4;          // then every piece starts on a 16-byte boundary
+    auto fetch = [&](int ch, float* dst) {
+        const int t0 = ch * DR_CH, nt = min(DR_CH, len - t0);
+        if (wide) {
+            const int nq = d >> 2, per = NV * nq + (ncol >> 2);
+            for (int i = threadIdx.x; i < nt * per; i += blockDim.x) {
+                const int t = i / per, k = i - t * per, r = r0 + t0 + t;
+                float* d0 = dst + t * PT;
+                if (k < nq) cp_async16s(d0 + dr_idx(4 * k, R), a.qn + ((size_t)r * Hk + hk) * d + 4 * k);
+                else if (k < 2 * nq) cp_async16s(d0 + DPD + dr_idx(4 * (k - nq), R), a.kn + ((size_t)r * Hk + hk) * d + 4 * (k - nq));
+                else if (PC && k < 3 * nq) cp_async16s(d0 + 2 * DPD + dr_idx(4 * (k - 2 * nq), R), a.dec + (size_t)r * a.lddec + h * d + 4 * (k - 2 * nq));
+                else cp_async16s(d0 + NV * DPD + 4 * (k - NV * nq), a.v + ((size_t)r * H + h) * dv + p0 + 4 * (k - NV * nq));
+            }
+        } else {
+            const int per = NV * d + ncol;
+            for (int i = threadIdx.x; i < nt * per; i += blockDim.x) {
+                const int t = i / per, k = i - t * per, r = r0 + t0 + t;
+                float* d0 = dst + t * PT;
+                if (k < d) cp_async4(d0 + dr_idx(k, R), a.qn + ((size_t)r * Hk + hk) * d + k);
+                else if (k < 2 * d) cp_async4(d0 + DPD + dr_idx(k - d, R), a.kn + ((size_t)r * Hk + hk) * d + k - d);
+                else if (PC && k < 3 * d) cp_async4(d0 + 2 * DPD + dr_idx(k - 2 * d, R), a.dec + (size_t)r * a.lddec + h * d + k - 2 * d);
+                else cp_async4(d0 + NV * DPD + k - NV * d, a.v + ((size_t)r * H + h) * dv + p0 + k - NV * d);
+            }
+        }
+        if (threadIdx.x < 3 * nt) {
+            const int t = threadIdx.x / 3, w = threadIdx.x % 3, r = r0 + t0 + t;
+            const float* src = w == 0 ? a.beta + (size_t)r * H + h : w == 1 ? a.qk + (size_t)r * Hk + hk : a.dec + (size_t)r * a.lddec + (PC ? h * d : h);
+            cp_async4(dst + t * PT + NV * DPD + DR_COLS + w, src);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        for (int t = nt; t < ((nt + 3) & ~3); ++t) {          // the last group's tokens past the end leave the state as it is
+            float* d0 = dst + t * PT;
+            if (PC) for (int i = threadIdx.x; i < DPD; i += blockDim.x) d0[2 * DPD + i] = 1.f;
+            if (threadIdx.x == 0) { d0[NV * DPD + DR_COLS] = 0.f; d0[NV * DPD + DR_COLS + 2] = 1.f; }
+        }
+    };
+    const int nch = (len + DR_CH - 1) / DR_CH;
+    fetch(0, stage[0]);
+    for (int ch = 0; ch < nch; ++ch) {
+        if (ch + 1 < nch) { fetch(ch + 1, stage[(ch + 1) & 1]); asm volatile("cp.async.wait_group 1;" ::: "memory"); }
+        else asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        const float* st = stage[ch & 1];
+        const int nt = min(DR_CH, len - ch * DR_CH);
+        for (int tg = 0; tg < nt; tg += 4) {
+            float o[4];
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                const float* tk = st + (tg + u) * PT;
+                float kk[R], qq[R];
+                load_run<R>(tk + dr_idx(n0, R), qq);
+                load_run<R>(tk + DPD + dr_idx(n0, R), kk);
+                const float4 sc = *reinterpret_cast<const float4*>(tk + NV * DPD + DR_COLS);      // step size, q . k, decay of the head
+                const float vv = tk[NV * DPD + pl];
+                float k0 = 0.f, k1 = 0.f, q0 = 0.f, q1 = 0.f;
+                if constexpr (PC) {
+                    float g[R];
+                    load_run<R>(tk + 2 * DPD + dr_idx(n0, R), g);
+#pragma unroll
+                    for (int i = 0; i < R; ++i) s[i] *= g[i];
+                }
+#pragma unroll
+                for (int i = 0; i < R; i += 2) {
+                    k0 = fmaf(s[i], kk[i], k0); q0 = fmaf(s[i], qq[i], q0);
+                    if (i + 1 < R) { k1 = fmaf(s[i + 1], kk[i + 1], k1); q1 = fmaf(s[i + 1], qq[i + 1], q1); }
+                }
+                float ks = k0 + k1, qs = q0 + q1;
+#pragma unroll
+                for (int m = DR_NS / 2; m > 0; m >>= 1) { ks += __shfl_xor_sync(0xffffffffu, ks, m); qs += __shfl_xor_sync(0xffffffffu, qs, m); }
+                const float dec = PC ? 1.f : sc.z, uu = sc.x * (vv - dec * ks);
+                if constexpr (PC) {
+#pragma unroll
+                    for (int i = 0; i < R; ++i) s[i] = fmaf(kk[i], uu, s[i]);
+                } else {
+#pragma unroll
+                    for (int i = 0; i < R; ++i) s[i] = fmaf(dec, s[i], kk[i] * uu);
+                }
+                o[u] = fmaf(sc.y, uu, dec * qs);
+            }
+            if (ns == 0) {
+#pragma unroll
+                for (int u = 0; u < 4; ++u) sy[(tg + u) * DR_COLS + pl] = o[u];
+            }
+        }
+        __syncthreads();
+        for (int i = threadIdx.x; i < nt * DR_COLS; i += blockDim.x) {
+            const int t = i / DR_COLS, c = i % DR_COLS;
+            if (c < ncol) a.y[((size_t)(r0 + ch * DR_CH + t) * H + h) * dv + p0 + c] = sy[i];
+        }
+        __syncthreads();                                      // the stage is free for chunk ch + 2
+    }
+#pragma unroll
+    for (int i = 0; i < R; ++i) if (live && n0 + i < d) S[(size_t)(n0 + i) * dv] = s[i];
+}
+
+// one warp per (row, head)
+__global__ void __launch_bounds__(128) delta_out_kernel(DeltaArgs a, int T) {
+    const int lane = threadIdx.x & 31, wid = blockIdx.x * 4 + (threadIdx.x >> 5);
+    if (wid >= T * a.H) return;
+    const int r = wid / a.H, h = wid % a.H, dv = a.dv;
+    const float* y = a.y + ((size_t)r * a.H + h) * dv;
+    const float* g = a.g + (size_t)r * a.ldg + h * dv;
+    float ss = 0.f;
+    for (int c = lane; c < dv; c += 32) ss = fmaf(y[c], y[c], ss);
+    const float inv = a.out_mult / sqrtf(warp_sum(ss) / (float)dv + a.eps);
+    for (int c = lane; c < dv; c += 32) store_act(a.out, r, a.out_col + h * dv + c, y[c] * inv * a.norm_w[c] * (a.gate_silu ? silu_f(g[c]) : sigmoid_f(g[c])));
+}
+
+// ---------------------------------------------------------------------------------------------------------------- the token's own embedding
+__global__ void token_gate_kernel(const float* __restrict__ z, int ldz, int n, const int* __restrict__ ids, const bf16* __restrict__ table, int ldt, int col0, ActOut out) {
+    const int r = blockIdx.y, j = blockIdx.x * blockDim.x + threadIdx.x;
+    if (j >= n) return;
+    store_act(out, r, j, gelu_tanh_f(z[(size_t)r * ldz + j]) * __bfloat162float(table[(size_t)ids[r] * ldt + col0 + j]));
+}
+// Block = (output j, row): 128 threads share the dot of length K, 16-byte loads of the bf16 weights.
+__global__ void __launch_bounds__(128) token_gate_step_kernel(const float* __restrict__ x, int ldx, const bf16* __restrict__ w, int ldw, int K, const int* __restrict__ ids,
+                                                              const bf16* __restrict__ table, int ldt, int col0, ActOut out) {
+    __shared__ float red[4];
+    const int j = blockIdx.x, r = blockIdx.y;
+    const uint4* w8 = reinterpret_cast<const uint4*>(w + (size_t)j * ldw);
+    const float4* x4 = reinterpret_cast<const float4*>(x + (size_t)r * ldx);
+    float acc = 0.f;
+    for (int k = threadIdx.x; k < K / 8; k += 128) {
+        const uint4 ww = w8[k];
+        const float4 a = x4[2 * k], b = x4[2 * k + 1];
+        acc = fmaf(bf16lo(ww.x), a.x, acc); acc = fmaf(bf16hi(ww.x), a.y, acc); acc = fmaf(bf16lo(ww.y), a.z, acc); acc = fmaf(bf16hi(ww.y), a.w, acc);
+        acc = fmaf(bf16lo(ww.z), b.x, acc); acc = fmaf(bf16hi(ww.z), b.y, acc); acc = fmaf(bf16lo(ww.w), b.z, acc); acc = fmaf(bf16hi(ww.w), b.w, acc);
+    }
+    acc = warp_sum(acc);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = acc;
+    __syncthreads();
+    if (threadIdx.x == 0) store_act(out, r, j, gelu_tanh_f((red[0] + red[1]) + (red[2] + red[3])) * __bfloat162float(table[(size_t)ids[r] * ldt + col0 + j]));
+}
+
+}  // namespace
+
+// ---------------------------------------------------------------------------------------------------------------- launchers
+int delta_launch_count(const DeltaArgs& a) { return 3 + (!a.single_rows && a.taps > 1 ? 1 : 0); }
+int delta_mixer_launch(cudaStream_t st, const RaggedBatch& rb, const DeltaArgs& a) {
+    if (a.d < 1 || a.d > 256 || a.dv < 1 || a.Hk < 1 || a.H % a.Hk || a.taps < 1 || !a.conv_w || (a.taps > 1 && !a.conv_state)) return -1000;
+    const int units = a.Hk + a.H + (a.per_channel ? a.H : 0) + 1, tile = a.single_rows ? 1 : rb.T >= 1024 ? DP_ROWS : 4, w = std::max(a.d, std::min(a.dv, 128));
+    const dim3 pgrid((rb.T + tile - 1) / tile, (units + 3) / 4);
+    auto prep = [&](auto k0, auto k1, auto k2, auto k3, auto k4) {
+        auto k = a.taps == 1 ? k1 : a.taps == 2 ? k2 : a.taps == 3 ? k3 : a.taps == 4 ? k4 : k0;
+        k<<<pgrid, 128, 0, st>>>(rb, a, tile);
+    };
+    if (w <= 64) prep(delta_prep_kernel<2, 0>, delta_prep_kernel<2, 1>, delta_prep_kernel<2, 2>, delta_prep_kernel<2, 3>, delta_prep_kernel<2, 4>);
+    else if (w <= 128) prep(delta_prep_kernel<4, 0>, delta_prep_kernel<4, 1>, delta_prep_kernel<4, 2>, delta_prep_kernel<4, 3>, delta_prep_kernel<4, 4>);
+    else prep(delta_prep_kernel<8, 0>, delta_prep_kernel<8, 1>, delta_prep_kernel<8, 2>, delta_prep_kernel<8, 3>, delta_prep_kernel<8, 4>);
+    int e = last_err();
+    if (e) return e;
+    if (!a.single_rows && a.taps > 1) {
+        CausalConvArgs ca = {};
+        ca.in = a.proj + a.col0; ca.ld = a.ld; ca.C = 2 * a.Hk * a.d + a.H * a.dv; ca.taps = a.taps; ca.state = a.conv_state;
+        if ((e = causal_conv_window_launch(st, rb, ca))) return e;
+    }
+    const int nr = (a.d + DR_NS - 1) / DR_NS, R = nr <= 2 ? 2 : nr <= 4 ? 4 : nr <= 8 ? 8 : nr <= 16 ? 16 : 32;
+    const size_t smem = (size_t)(2 * DR_CH * ((a.per_channel ? 3 : 2) * dr_pad(R) + DR_COLS + 4) + DR_CH * DR_COLS) * sizeof(float);      // <= 113 KB at d = 256
+    static SmemOptIn seen[2][5];
+    auto run = [&](auto kern, SmemOptIn& s) -> int {
+        if (const int er = ensure_dyn_smem(kern, smem, s)) return er;
+        kern<<<dim3(rb.E, a.H, (a.dv + DR_COLS - 1) / DR_COLS), DR_COLS * DR_NS, smem, st>>>(rb, a);
+        return last_err();
+    };
+    if (a.per_channel) e = R == 2 ? run(delta_scan_kernel<2, true>, seen[1][0]) : R == 4 ? run(delta_scan_kernel<4, true>, seen[1][1]) : R == 8 ? run(delta_scan_kernel<8, true>, seen[1][2])
+                         : R == 16 ? run(delta_scan_kernel<16, true>, seen[1][3]) : run(delta_scan_kernel<32, true>, seen[1][4]);
+    else e = R == 2 ? run(delta_scan_kernel<2, false>, seen[0][0]) : R == 4 ? run(delta_scan_kernel<4, false>, seen[0][1]) : R == 8 ? run(delta_scan_kernel<8, false>, seen[0][2])
+           : R == 16 ? run(delta_scan_kernel<16, false>, seen[0][3]) : run(delta_scan_kernel<32, false>, seen[0][4]);
+    if (e) return e;
+    delta_out_kernel<<<(rb.T * a.H + 3) / 4, 128, 0, st>>>(a, rb.T);
+    return last_err();
+}
+int token_gate_launch(cudaStream_t st, const float* z, int ldz, int T, int n, const int* ids, const bf16* table, int ldt, int col0, const ActOut& out) {
+    if (n < 1) return -1000;
+    token_gate_kernel<<<dim3((n + 127) / 128, T), 128, 0, st>>>(z, ldz, n, ids, table, ldt, col0, out);
+    return last_err();
+}
+int token_gate_step_launch(cudaStream_t st, const float* x, int ldx, const bf16* w, int ldw, int K, int T, int n, const int* ids, const bf16* table, int ldt,
+                           int col0, const ActOut& out) {
+    if (n < 1 || (K & 7) || (ldw & 7) || (ldx & 3)) return -1000;
+    token_gate_step_kernel<<<dim3(n, T), 128, 0, st>>>(x, ldx, w, ldw, K, ids, table, ldt, col0, out);
+    return last_err();
+}
+
+}  // namespace cb

@@ -450,6 +450,11 @@ int causal_conv_launch(cudaStream_t st, const RaggedBatch& rb, const CausalConvA
     if (a.taps > 1) causal_conv_window_kernel<<<dim3((a.C + 127) / 128, rb.E), 128, 0, st>>>(rb, a);
     return last_err();
 }
+int causal_conv_window_launch(cudaStream_t st, const RaggedBatch& rb, const CausalConvArgs& a) {
+    if (a.taps < 2 || a.C < 1 || !a.in || !a.state) return -1000;
+    causal_conv_window_kernel<<<dim3((a.C + 127) / 128, rb.E), 128, 0, st>>>(rb, a);
+    return last_err();
+}
 bool norm_conv_step_fits(int W, int groups, int taps) { return groups >= 1 && groups <= NCS_GROUPS && W % groups == 0 && taps >= 1 && taps <= 4 && W <= 1024 * NCS_COLS; }
 int norm_conv_step_launch(cudaStream_t st, const RaggedBatch& rb, const float* x, int ldx, int W, int groups, float eps, const float* norm_w,
                           int taps, const float* conv_w, float* state, const ActOut& out_h, const ActOut& out_u) {
