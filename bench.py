@@ -699,6 +699,77 @@ def bench_nifarax(args, rank, world, local_rank):
     print(json.dumps(out))
 
 
+def layer_list_load(cls, cfg, S, n_dec):
+    """A layer-list model with random weights: big matrices as random bf16 blocks (timing only), the small tensors drawn properly."""
+    import crane_b200  # noqa: F401
+    sys.path.insert(0, os.path.join(ROOT, "tools"))
+    import bench_configs as bc
+    m = cls(cfg, device=0, max_tokens=S + n_dec + 128, max_batch=4)
+    for name, shape, kind in synth.tensor_specs(cfg):
+        big = len(shape) == 2 and shape[0] * shape[1] >= (1 << 18) and kind in ("linear", "embed")
+        m.load_tensor(name, bc.cheap(shape, kind) if big else synth.make_tensor(name, shape, kind))
+    m.finalize()
+    return m
+
+
+def layer_list_work(cfg, S, n_dec):
+    """(weights a token touches, attention / recurrence flops of the prompt, bytes of cache and state a decode step touches)"""
+    W, V = cfg["width"], cfg["vocab"]
+    shapes = {n: sh for n, sh, k in synth.tensor_specs(cfg)}
+    per_tok, attn_fl, cache_b = V * W, 0.0, 0.0
+    for i, L in enumerate(cfg["layers"]):
+        per_tok += sum(sh[0] * sh[1] for n, sh in shapes.items() if n.startswith(f"l{i}.") and len(sh) == 2 and ".mix.conv" not in n and not n.endswith(".conv"))
+        a = L["mixer"]
+
+        def attention(a):
+            keys = min(S / 2, a["mask"]["size"]) if a.get("mask") else S / 2
+            ctx = min(S + n_dec / 2, a["mask"]["size"]) if a.get("mask") else S + n_dec / 2
+            return 2.0 * S * keys * a["heads"] * (a["dim"] + a["vdim"]), ctx * a["kv_heads"] * (a["dim"] + a["vdim"]) * 4
+        if L["type"] == "attention":
+            f, b = attention(a)
+        elif L["type"] == "parallel":
+            f, b = attention(a["left"])
+            r = a["right"]
+            f += (6.0 if "conv" in r else 4.0) * S * r["heads"] * r["dim"] * r["vdim"]      # (the delta rule takes a third product with the state)
+            b += 2 * 4 * r["heads"] * r["dim"] * r["vdim"]
+        elif L["type"] == "delta":
+            f, b = 6.0 * S * a["heads"] * a["dim"] * a["vdim"], 2 * 4 * a["heads"] * a["dim"] * a["vdim"]
+        elif L["type"] == "mamba1":
+            f, b = 6.0 * S * a["inner"] * a["state"], 2 * 4 * a["inner"] * a["state"]
+        else:
+            f, b = 4.0 * S * a["heads"] * a["state"] * a["vdim"], 2 * 4 * a["heads"] * a["state"] * a["vdim"]
+        attn_fl += f
+        cache_b += b
+    return per_tok, attn_fl, cache_b
+
+
+def layer_list_measure(m, cfg, tag, args, peaks, S, n_dec):
+    ids = synth.synth_token_ids(S, cfg["vocab"], tag)
+
+    def request():
+        m.clear_kv_cache()
+        t0 = time.perf_counter()
+        out = m.generate_greedy(ids, n_dec + 1)
+        wall = time.perf_counter() - t0
+        t = m.last_timing()
+        return wall, t["prefill_ms"], t["decode_ms"], len(out) - 1
+    for _ in range(max(args.warmup, 3)):
+        request()
+    l0 = m.kernel_launches()
+    rs = [request() for _ in range(args.steps)]
+    launches = m.kernel_launches() - l0
+    per_tok, attn_fl, cache_b = layer_list_work(cfg, S, n_dec)
+    W, V = cfg["width"], cfg["vocab"]
+    fl = 2.0 * (per_tok - V * W) * S + attn_fl + 2.0 * V * W
+    by = 2.0 * per_tok + cache_b
+    dec_s, ntok, pre_s = sum(r[2] for r in rs) / 1e3, sum(r[3] for r in rs), sum(r[1] for r in rs) / 1e3
+    return {"decode_tok_s": ntok / dec_s, "decode_us_per_step": 1e6 * dec_s / ntok, "prefill_ms": 1e3 * pre_s / len(rs),
+            "prefill_tok_s": S * len(rs) / pre_s, "prefill_tflops": fl * len(rs) / pre_s / 1e12,
+            "prefill_frac_of_bf16_peak": fl * len(rs) / pre_s / 1e12 / peaks["bf16_tflops"],
+            "decode_hbm_gbs": by / (dec_s / ntok) / 1e9, "decode_roofline_frac": by / (dec_s / ntok) / 1e9 / peaks["hbm_gbs"],
+            "algorithmic_bytes_per_step": by, "prefill_flop": fl, "e2e_tok_s": ntok / sum(r[0] for r in rs), "gpu_launches": int(launches)}
+
+
 def bench_puzonex(args, rank, world, local_rank):
     """The Puzonex layer-list decoder (sublayers normalised on their way back; Mamba-1, capped sink attention with a distance penalty,
     windowed attention beside a matrix memory; tanh-GELU gated feed-forward) beside the closest existing model, a Fosovik stack with
@@ -706,8 +777,6 @@ def bench_puzonex(args, rank, world, local_rank):
     width, depth, heads and feed-forward width, at two sizes.  One request = 4096-token prefill + 256 greedy tokens through
     `crane_b200_generate_greedy`; random bf16 blocks as weights (timing only; the small tensors are drawn properly); one GPU."""
     import crane_b200
-    sys.path.insert(0, os.path.join(ROOT, "tools"))
-    import bench_configs as bc
     if args.impl == "reference":
         if rank == 0:
             print(json.dumps({"impl": "reference", "unavailable": "the reference has no model of this design"}))
@@ -735,68 +804,6 @@ def bench_puzonex(args, rank, world, local_rank):
             fsv=closest(2048, 9, 16, 4, 128, 32, 128, 16, 5632)),
     }
 
-    def load(cls, cfg):
-        m = cls(cfg, device=0, max_tokens=S + n_dec + 128, max_batch=4)
-        for name, shape, kind in synth.tensor_specs(cfg):
-            big = len(shape) == 2 and shape[0] * shape[1] >= (1 << 18) and kind in ("linear", "embed")
-            m.load_tensor(name, bc.cheap(shape, kind) if big else synth.make_tensor(name, shape, kind))
-        m.finalize()
-        return m
-
-    def work(cfg):
-        """(weights a token touches, attention / recurrence flops of the prompt, bytes of cache and state a decode step touches)"""
-        W, V = cfg["width"], cfg["vocab"]
-        shapes = {n: sh for n, sh, k in synth.tensor_specs(cfg)}
-        per_tok, attn_fl, cache_b = V * W, 0.0, 0.0
-        for i, L in enumerate(cfg["layers"]):
-            per_tok += sum(sh[0] * sh[1] for n, sh in shapes.items() if n.startswith(f"l{i}.") and len(sh) == 2 and ".mix.conv" not in n)
-            a = L["mixer"]
-
-            def attention(a):
-                keys = min(S / 2, a["mask"]["size"]) if a.get("mask") else S / 2
-                ctx = min(S + n_dec / 2, a["mask"]["size"]) if a.get("mask") else S + n_dec / 2
-                return 2.0 * S * keys * a["heads"] * (a["dim"] + a["vdim"]), ctx * a["kv_heads"] * (a["dim"] + a["vdim"]) * 4
-            if L["type"] == "attention":
-                f, b = attention(a)
-            elif L["type"] == "parallel":
-                f, b = attention(a["left"])
-                r = a["right"]
-                f += 4.0 * S * r["heads"] * r["dim"] * r["vdim"]
-                b += 2 * 4 * r["heads"] * r["dim"] * r["vdim"]
-            elif L["type"] == "mamba1":
-                f, b = 6.0 * S * a["inner"] * a["state"], 2 * 4 * a["inner"] * a["state"]
-            else:
-                f, b = 4.0 * S * a["heads"] * a["state"] * a["vdim"], 2 * 4 * a["heads"] * a["state"] * a["vdim"]
-            attn_fl += f
-            cache_b += b
-        return per_tok, attn_fl, cache_b
-
-    def measure(m, cfg, tag):
-        ids = synth.synth_token_ids(S, cfg["vocab"], tag)
-
-        def request():
-            m.clear_kv_cache()
-            t0 = time.perf_counter()
-            out = m.generate_greedy(ids, n_dec + 1)
-            wall = time.perf_counter() - t0
-            t = m.last_timing()
-            return wall, t["prefill_ms"], t["decode_ms"], len(out) - 1
-        for _ in range(max(args.warmup, 3)):
-            request()
-        l0 = m.kernel_launches()
-        rs = [request() for _ in range(args.steps)]
-        launches = m.kernel_launches() - l0
-        per_tok, attn_fl, cache_b = work(cfg)
-        W, V = cfg["width"], cfg["vocab"]
-        fl = 2.0 * (per_tok - V * W) * S + attn_fl + 2.0 * V * W
-        by = 2.0 * per_tok + cache_b
-        dec_s, ntok, pre_s = sum(r[2] for r in rs) / 1e3, sum(r[3] for r in rs), sum(r[1] for r in rs) / 1e3
-        return {"decode_tok_s": ntok / dec_s, "decode_us_per_step": 1e6 * dec_s / ntok, "prefill_ms": 1e3 * pre_s / len(rs),
-                "prefill_tok_s": S * len(rs) / pre_s, "prefill_tflops": fl * len(rs) / pre_s / 1e12,
-                "prefill_frac_of_bf16_peak": fl * len(rs) / pre_s / 1e12 / peaks["bf16_tflops"],
-                "decode_hbm_gbs": by / (dec_s / ntok) / 1e9, "decode_roofline_frac": by / (dec_s / ntok) / 1e9 / peaks["hbm_gbs"],
-                "algorithmic_bytes_per_step": by, "prefill_flop": fl, "e2e_tok_s": ntok / sum(r[0] for r in rs), "gpu_launches": int(launches)}
-
     only = os.environ.get("CRANE_B200_BENCH_ONLY", "")          # "puzonex" / "closest": one side only (launch lists, profiles)
     variants = {}
     sampler.start()
@@ -806,8 +813,8 @@ def bench_puzonex(args, rank, world, local_rank):
             if only and not key.startswith(only):
                 continue
             cfg = pair["pzx" if key == "puzonex" else "fsv"]
-            m = load(cls, cfg)
-            variants[name][key] = measure(m, cfg, name + key)
+            m = layer_list_load(cls, cfg, S, n_dec)
+            variants[name][key] = layer_list_measure(m, cfg, name + key, args, peaks, S, n_dec)
             m.close()
         if only:
             break
@@ -817,6 +824,72 @@ def bench_puzonex(args, rank, world, local_rank):
     out = {"metric": "decode_tok_per_s", "unit": "tok/s", "n_gpus": 1, "steps": args.steps, "warmup": max(args.warmup, 3), "higher_is_better": True,
            "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
            "config": {"workload": f"Puzonex layer-list decoder (width 1024, 4 x (Mamba-1, attention beside a matrix memory, attention), window 1024, feed-forward 3584), {S}-token prefill + {n_dec} greedy decode tokens per request; the closest existing model at equal size beside it",
+                      "weights": "random bf16 blocks (timing only)", "l2": "per-token weight stream > 126 MB L2", "parallelism": "1 GPU",
+                      "precision": os.environ.get("CRANE_B200_PRECISION", "split")},
+           "value": d["decode_tok_s"], "ms_per_step": 1e3 / d["e2e_tok_s"] * n_dec, "prefill_ms": d["prefill_ms"], "prefill_tflops": d["prefill_tflops"],
+           "e2e": {"value": d["e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": int(S * 4), "d2h_bytes_per_step": int((n_dec + 1) * 4),
+                   "api": "crane_b200_generate_greedy (host prompt ids in, host token ids out; prefill inside the timed region)"},
+           "gpu_launches": d["gpu_launches"], "clocks": clocks, "variants": variants,
+           "roofline": {"bound": "hbm", "achieved": d["decode_hbm_gbs"], "peak": peaks["hbm_gbs"], "unit": "GB/s", "frac": d["decode_roofline_frac"],
+                        "peak_source": peaks["source"], "launch": "one decode step (graph replay): the token's weights once + the windows' cached keys and values + recurrent states"}}
+    print(json.dumps(out))
+
+
+def bench_suvapel(args, rank, world, local_rank):
+    """The Suvapel layer-list decoder (Dynamic-Tanh layers with a joint residual: the gated delta rule, windowed attention with kept first
+    tokens beside a delta rule with a decay per key channel, a SiLU-gated feed-forward, a token embedding behind every layer) beside the
+    closest existing model, a Puzonex stack with Mamba-1 where Suvapel has the delta rule alone and windowed attention beside a matrix
+    memory (of the same state size) where it has its parallel mixer, at equal width, depth, heads and feed-forward width, at two sizes.
+    One request = 4096-token prefill + 256 greedy tokens through `crane_b200_generate_greedy`; one GPU."""
+    if args.impl == "reference":
+        if rank == 0:
+            print(json.dumps({"impl": "reference", "unavailable": "the reference has no model of this design"}))
+        return
+    if rank != 0:
+        return
+    import crane_b200
+    S, n_dec = 4096, 256
+    peaks = load_peaks()
+    sampler = ClockSampler(0)
+
+    def closest(**kw):
+        c = synth.puzonex_config(**kw)
+        rec, par, _ = c["layers"][:3]
+        c["layers"] = [dict(rec) if i % 3 == 0 else dict(par) for i in range(len(c["layers"]))]
+        return c
+    sizes = {
+        "w1024_12layers_ff3584": dict(
+            svp=synth.suvapel_config(width=1024, layers=12, heads=8, kv_heads=2, dim=128, window=1024, r_heads=8, r_dim=128, ff=3584, rank=128, side=128),
+            pzx=closest(width=1024, layers=12, heads=8, kv_heads=2, dim=128, window=1024, inner=2048, state=16, dt_rank=64, mem_heads=4, mem_dim=128,
+                        mem_vdim=256, ff=3584)),
+        "w2048_9layers_ff5632": dict(
+            svp=synth.suvapel_config(width=2048, layers=9, heads=16, kv_heads=4, dim=128, window=2048, r_heads=16, r_dim=128, ff=5632, rank=128, side=256),
+            pzx=closest(width=2048, layers=9, heads=16, kv_heads=4, dim=128, window=2048, inner=4096, state=16, dt_rank=128, mem_heads=8, mem_dim=128,
+                        mem_vdim=256, bias_max=2048, ff=5632)),
+    }
+    only = os.environ.get("CRANE_B200_BENCH_ONLY", "")          # "suvapel" / "closest": one side only (launch lists, profiles)
+    cut = int(os.environ.get("CRANE_B200_BENCH_LAYERS", "0"))   # with it: that many layers only
+    variants = {}
+    sampler.start()
+    for name, pair in sizes.items():
+        variants[name] = {}
+        for key, cls in (("suvapel", crane_b200.SuvapelModel), ("closest_model_puzonex", crane_b200.PuzonexModel)):
+            if only and not key.startswith(only):
+                continue
+            cfg = pair["svp" if key == "suvapel" else "pzx"]
+            if only and cut:
+                cfg["layers"] = cfg["layers"][:cut]
+            m = layer_list_load(cls, cfg, S, n_dec)
+            variants[name][key] = layer_list_measure(m, cfg, name + key, args, peaks, S, n_dec)
+            m.close()
+        if only:
+            break
+    clocks = sampler.summary()
+    first = variants["w1024_12layers_ff3584"]
+    d = first.get("suvapel") or first["closest_model_puzonex"]
+    out = {"metric": "decode_tok_per_s", "unit": "tok/s", "n_gpus": 1, "steps": args.steps, "warmup": max(args.warmup, 3), "higher_is_better": True,
+           "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+           "config": {"workload": f"Suvapel layer-list decoder (width 1024, 4 x (delta rule, 2 x (attention beside a delta rule)), window 1024, feed-forward 3584), {S}-token prefill + {n_dec} greedy decode tokens per request; the closest existing model at equal size beside it",
                       "weights": "random bf16 blocks (timing only)", "l2": "per-token weight stream > 126 MB L2", "parallelism": "1 GPU",
                       "precision": os.environ.get("CRANE_B200_PRECISION", "split")},
            "value": d["decode_tok_s"], "ms_per_step": 1e3 / d["e2e_tok_s"] * n_dec, "prefill_ms": d["prefill_ms"], "prefill_tflops": d["prefill_tflops"],
@@ -856,7 +929,7 @@ def main():
     ap.add_argument("--steps", type=int, default=5)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="crane_b200", choices=["crane_b200", "reference"])
-    ap.add_argument("--config", default="qwen3_vl_2b", choices=["qwen3_vl_2b", "tiny", "qwen3_8b_q4km", "qwen3_5_0_8b", "fosovik", "gavipel", "nifarax", "puzonex"])
+    ap.add_argument("--config", default="qwen3_vl_2b", choices=["qwen3_vl_2b", "tiny", "qwen3_8b_q4km", "qwen3_5_0_8b", "fosovik", "gavipel", "nifarax", "puzonex", "suvapel"])
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-other-configs", action="store_true", help="skip the config-2 (Qwen3.5-0.8B) child measurement appended to the headline line")
     args = ap.parse_args()
@@ -876,6 +949,8 @@ def main():
         return bench_nifarax(args, rank, world, local_rank)
     if args.config == "puzonex":
         return bench_puzonex(args, rank, world, local_rank)
+    if args.config == "suvapel":
+        return bench_suvapel(args, rank, world, local_rank)
     cfg = synth.QWEN3_VL_2B if args.config == "qwen3_vl_2b" else synth.TINY_QWEN3_VL
     name = "Qwen3-VL-2B" if args.config == "qwen3_vl_2b" else "tiny-Qwen3-VL"
     workload = f"{name} bf16, 1x(448x448) image + {N_TEXT}-tok prompt, prefill + {N_DECODE} greedy decode tokens per request"

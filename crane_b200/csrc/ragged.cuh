@@ -337,7 +337,13 @@ struct DeltaArgs {
     float* dec; int lddec;            // scratch [T, lddec] for the decays, H*d or H columns (per channel: may be z itself)
     ActOut out; int out_col;          // [T, .. out_col + H*dv]
     int max_len = 0;                  // rows of the longest entry
+    // portions from DELTA_CHUNK_MIN rows on go 16 tokens at a time (ragged_delta_chunk.cu): scratch of delta_chunk_ws_floats(T, E, ...)
+    // floats; nullptr = always token by token, every product and sum in f32 on CUDA cores
+    float* chunk_ws = nullptr;
 };
+constexpr int DELTA_CHUNK_MIN = 48;
+size_t delta_chunk_ws_floats(int rows, int entries, int H, int d, int dv);
+int delta_chunk_launch(cudaStream_t st, const RaggedBatch& rb, const DeltaArgs& a);
 int delta_mixer_launch(cudaStream_t st, const RaggedBatch& rb, const DeltaArgs& a);
 int delta_launch_count(const DeltaArgs& a);
 

@@ -1,7 +1,7 @@
 // The gated delta rule on ragged batches (see ragged.cuh), and the embedding of the token that joins behind a layer.
 //   prep : per (q / k head | value head | gates): convolution over time with the carried window, SiLU, unit norms, q . k, the decays
 //          and step sizes -- f32 throughout, one warp per head and tile of rows, the tap window in registers;
-//   scan : the recurrence token by token, a thread keeps its share of the state in registers for the whole portion, the inputs of
+//   scan : the recurrence token by token (long portions: 16 tokens at a time, ragged_delta_chunk.cu), a thread keeps its share of the state in registers for the whole portion, the inputs of
 //          DR_CH tokens at a time staged in shared memory (cp.async, double-buffered);
 //   out  : norm over the value width, gate.
 // A row's result depends on its own sequence only: the split of the state over lanes and the order of the lane sums are launch
@@ -344,7 +344,8 @@ __global__ void __launch_bounds__(128) token_gate_step_kernel(const float* __res
 }  // namespace
 
 // ---------------------------------------------------------------------------------------------------------------- launchers
-int delta_launch_count(const DeltaArgs& a) { return 3 + (!a.single_rows && a.taps > 1 ? 1 : 0); }
+static bool by_chunks(const DeltaArgs& a) { return a.chunk_ws && a.max_len >= DELTA_CHUNK_MIN; }
+int delta_launch_count(const DeltaArgs& a) { return 3 + (!a.single_rows && a.taps > 1 ? 1 : 0) + (by_chunks(a) ? 1 : 0); }
 int delta_mixer_launch(cudaStream_t st, const RaggedBatch& rb, const DeltaArgs& a) {
     if (a.d < 1 || a.d > 256 || a.dv < 1 || a.Hk < 1 || a.H % a.Hk || a.taps < 1 || !a.conv_w || (a.taps > 1 && !a.conv_state)) return -1000;
     const int units = a.Hk + a.H + (a.per_channel ? a.H : 0) + 1, tile = a.single_rows ? 1 : rb.T >= 1024 ? DP_ROWS : 4, w = std::max(a.d, std::min(a.dv, 128));
@@ -371,7 +372,8 @@ int delta_mixer_launch(cudaStream_t st, const RaggedBatch& rb, const DeltaArgs& 
         kern<<<dim3(rb.E, a.H, (a.dv + DR_COLS - 1) / DR_COLS), DR_COLS * DR_NS, smem, st>>>(rb, a);
         return last_err();
     };
-    if (a.per_channel) e = R == 2 ? run(delta_scan_kernel<2, true>, seen[1][0]) : R == 4 ? run(delta_scan_kernel<4, true>, seen[1][1]) : R == 8 ? run(delta_scan_kernel<8, true>, seen[1][2])
+    if (by_chunks(a)) e = delta_chunk_launch(st, rb, a);
+    else if (a.per_channel) e = R == 2 ? run(delta_scan_kernel<2, true>, seen[1][0]) : R == 4 ? run(delta_scan_kernel<4, true>, seen[1][1]) : R == 8 ? run(delta_scan_kernel<8, true>, seen[1][2])
                          : R == 16 ? run(delta_scan_kernel<16, true>, seen[1][3]) : run(delta_scan_kernel<32, true>, seen[1][4]);
     else e = R == 2 ? run(delta_scan_kernel<2, false>, seen[0][0]) : R == 4 ? run(delta_scan_kernel<4, false>, seen[0][1]) : R == 8 ? run(delta_scan_kernel<8, false>, seen[0][2])
            : R == 16 ? run(delta_scan_kernel<16, false>, seen[0][3]) : run(delta_scan_kernel<32, false>, seen[0][4]);

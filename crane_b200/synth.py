@@ -605,7 +605,80 @@ def puzonex_tensor_specs(cfg: dict):
     yield "head", (V, W), "embed"
 
 
+def suvapel_config(width=1024, vocab=65536, layers=12, heads=8, kv_heads=2, dim=128, window=1024, keep_first=4, r_heads=8, r_dim=128, conv=4, rank=128,
+                   side=128, ff=3584):
+    """`layers` layers in the order delta rule, attention beside a delta rule, attention beside a delta rule, ..., each with a SiLU-gated
+    feed-forward.  `a_rank` / `g_rank` are not read by the engine (ranks come with the tensors); they tell `suvapel_tensor_specs` which
+    shapes to make."""
+    rule = {"heads": r_heads, "kv_heads": r_heads, "dim": r_dim, "vdim": r_dim, "conv": conv}
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "conv": conv, "mask": {"size": window, "keep_first": keep_first}, "scale": dim ** -0.5,
+            "rot": {"base": 500000.0, "dims": dim // 2, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    par = {"left": left, "right": dict(rule, a_rank=rank, g_rank=rank), "left_scale": 0.5, "right_scale": 0.5}
+    mlp = {"kind": "dense", "ff": ff} if ff else None
+    ls = [{"type": "delta" if i % 3 == 0 else "parallel", "mixer": dict(rule if i % 3 == 0 else par), "mlp": dict(mlp) if mlp else None} for i in range(layers)]
+    return {"architecture": "Suvapel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "token_side": {"dim": side}, "layers": ls}
+
+
+def suvapel_tensor_specs(cfg: dict):
+    """(name, shape, kind): 'embed', 'side.embed', 'final.norm[.b|.alpha]', 'head', 'l<i>.norm1[.b|.alpha]', 'l<i>.mlp.gate|up|down[.b]',
+    'l<i>.side.gate|proj|norm', and per mixer 'l<i>.mix.q|k|v[.conv]|b|a|g|A_log|dt_bias|norm|o', or 'l<i>.mix.left.q|k|v[.conv]|g|o' with
+    'l<i>.mix.right.q|k|v[.conv]|b|a1|a2|g1|g2|A_log|dt_bias|norm|o'."""
+    W, V, sd = cfg["width"], cfg["vocab"], cfg["token_side"]["dim"]
+    yield "embed", (V, W), "embed"
+    yield "side.embed", (V, sd * len(cfg["layers"])), "embed"
+
+    def rule(p, m, low_rank):
+        H, Hk, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        for t, n in (("q", Hk * d), ("k", Hk * d), ("v", H * dv)):
+            yield p + t, (n, W), "linear"
+            yield p + t + ".conv", (n, m["conv"]), "linear"
+        yield p + "b", (H, W), "linear"
+        yield p + "A_log", (H,), "a_log"
+        if low_rank:
+            ra, rg = m.get("a_rank", 128), m.get("g_rank", 128)
+            yield p + "a1", (ra, W), "linear"
+            yield p + "a2", (H * d, ra), "linear"
+            yield p + "g1", (rg, W), "linear"
+            yield p + "g2", (H * dv, rg), "linear"
+        else:
+            yield p + "a", (H, W), "linear"
+            yield p + "g", (H * dv, W), "linear"
+        yield p + "dt_bias", (H * d if low_rank else H,), "dt_bias"
+        yield p + "norm", (dv,), "norm"
+        yield p + "o", (W, H * dv), "linear"
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        yield p + "norm1", (W,), "norm"
+        yield p + "norm1.b", (W,), "bias"
+        yield p + "norm1.alpha", (1,), "norm"
+        if L["type"] == "parallel":
+            a = m["left"]
+            for t, n in (("q", a["heads"] * a["dim"]), ("k", a["kv_heads"] * a["dim"]), ("v", a["kv_heads"] * a["vdim"])):
+                yield p + "mix.left." + t, (n, W), "linear"
+                yield p + "mix.left." + t + ".conv", (n, a["conv"]), "linear"
+            yield p + "mix.left.g", (a["heads"], W), "linear"
+            yield p + "mix.left.o", (W, a["heads"] * a["vdim"]), "linear"
+            yield from rule(p + "mix.right.", m["right"], True)
+        else:
+            yield from rule(p + "mix.", m, False)
+        if L.get("mlp"):
+            F = L["mlp"]["ff"]
+            for t, sh in (("gate", (F, W)), ("up", (F, W)), ("down", (W, F))):
+                yield p + "mlp." + t, sh, "linear"
+                yield p + "mlp." + t + ".b", (sh[0],), "bias"
+        yield p + "side.gate", (sd, W), "linear"
+        yield p + "side.proj", (W, sd), "linear"
+        yield p + "side.norm", (W,), "norm"
+    yield "final.norm", (W,), "norm"
+    yield "final.norm.b", (W,), "bias"
+    yield "final.norm.alpha", (1,), "norm"
+    yield "head", (V, W), "embed"
+
+
 def tensor_specs(cfg: dict):
+    if cfg.get("architecture") == "Suvapel":
+        yield from suvapel_tensor_specs(cfg)
+        return
     if cfg.get("architecture") == "Puzonex":
         yield from puzonex_tensor_specs(cfg)
         return
