@@ -132,14 +132,14 @@ __device__ __forceinline__ void epi_block(const GemmEpi& ep, uint8_t* stg, int m
     if (ep.bias != nullptr) {
 #pragma unroll
         for (int j = 0; j < 32; j += 4) {
-            const float4 b = *reinterpret_cast<const float4*>(ep.bias + n + j);
+            const float4 b = __ldg(reinterpret_cast<const float4*>(ep.bias + n + j));
             v[j] += b.x; v[j + 1] += b.y; v[j + 2] += b.z; v[j + 3] += b.w;
         }
     }
     if (ep.col_scale != nullptr) {
 #pragma unroll
         for (int j = 0; j < 32; j += 4) {
-            const float4 c = *reinterpret_cast<const float4*>(ep.col_scale + n + j);
+            const float4 c = __ldg(reinterpret_cast<const float4*>(ep.col_scale + n + j));
             v[j] *= c.x; v[j + 1] *= c.y; v[j + 2] *= c.z; v[j + 3] *= c.w;
         }
     }

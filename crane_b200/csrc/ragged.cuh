@@ -340,12 +340,18 @@ struct DeltaArgs {
     // portions from DELTA_CHUNK_MIN rows on go 16 tokens at a time (ragged_delta_chunk.cu): scratch of delta_chunk_ws_floats(T, E, ...)
     // floats; nullptr = always token by token, every product and sum in f32 on CUDA cores
     float* chunk_ws = nullptr;
+    // delta_step_launch only: the second factors of low-rank decays and gates ([H*d, ld_a2], [H*dv, ld_g2] bf16, zeros behind the ranks),
+    // multiplied in the launch itself by the first factors in proj's columns a_col .. / g_col ..; nullptr = z and g are given
+    const bf16 *w_a2 = nullptr, *w_g2 = nullptr; int ld_a2 = 0, ld_g2 = 0, a_col = 0, g_col = 0, a_rank = 0, g_rank = 0;
 };
 constexpr int DELTA_CHUNK_MIN = 48;
 size_t delta_chunk_ws_floats(int rows, int entries, int H, int d, int dv);
 int delta_chunk_launch(cudaStream_t st, const RaggedBatch& rb, const DeltaArgs& a);
 int delta_mixer_launch(cudaStream_t st, const RaggedBatch& rb, const DeltaArgs& a);
 int delta_launch_count(const DeltaArgs& a);
+// every entry one row: all of the mixer in one launch, for the sizes delta_step_fits() accepts (the others take delta_mixer_launch)
+bool delta_step_fits(int H, int Hk, int d, int dv, int taps);
+int delta_step_launch(cudaStream_t st, const RaggedBatch& rb, const DeltaArgs& a);
 
 // A token's own embedding behind a layer: out[r, j] = gelu_tanh(z[r, j]) * table[ids[r], col0 + j], j < n (table [V, ldt] bf16)
 int token_gate_launch(cudaStream_t st, const float* z, int ldz, int T, int n, const int* ids, const bf16* table, int ldt, int col0, const ActOut& out);

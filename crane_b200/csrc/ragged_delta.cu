@@ -315,6 +315,150 @@ __global__ void __launch_bounds__(128) delta_out_kernel(DeltaArgs a, int T) {
     for (int c = lane; c < dv; c += 32) store_act(a.out, r, a.out_col + h * dv + c, y[c] * inv * a.norm_w[c] * (a.gate_silu ? silu_f(g[c]) : sigmoid_f(g[c])));
 }
 
+// ---------------------------------------------------------------------------------------------------------------- a decode step
+// Every entry one row: the whole mixer between the merged projection and the output projection in one launch.  Block = (head, 32 value
+// columns, entry); the blocks of the heads that share a q / k head form a cluster.  Convolution and unit norms (every block for itself), the
+// low-rank products (w_a2 != nullptr: z and the gate's pre-activations are taken here from the first factors in proj; a head's blocks
+// share the decays' rows and hand the results round), decays and step size; then the state, read once and written once, a thread owning
+// R rows of one column; norm over the head's blocks, gate.  The windows move on after every block of the cluster has read them.
+constexpr int DS_NS = 8, DS_TAPS = 8, DS_NT = DS_NS * 32, DS_CONV = 3;      // row slices, most taps, threads, channels per thread at most
+__device__ __forceinline__ void cluster_store(float* p, int rank, float v) {     // to the same place in another block of the cluster
+    uint32_t a;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(a) : "r"(smem_u32(p)), "r"(rank));
+    asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(a), "f"(v) : "memory");
+}
+__device__ __forceinline__ void cluster_sync() {
+    asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
+    asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+template <int R>
+__global__ void __launch_bounds__(DS_NT, 1) delta_step_kernel(RaggedBatch rb, DeltaArgs a) {
+    extern __shared__ __align__(16) float xs[];           // the first factors' outputs (low-rank form)
+    constexpr int DR = DS_NS * R;
+    __shared__ __align__(16) float sq[DR], sk[DR], sdec[DR], sv[32], sg[32], part[2][DS_NS][32], sz[DR + 32];
+    __shared__ float scal[3], ssum[8];                    // 1 / |q| (with q_scale), 1 / |k|, their product before the norms; the blocks' sums of squares
+    const int d = a.d, dv = a.dv, H = a.H, Hk = a.Hk, rep = H / Hk, nz = (dv + 31) / 32, h = blockIdx.x / nz, z = blockIdx.x % nz, e = blockIdx.y;
+    const int hk = h / rep, C = 2 * Hk * d + H * dv, taps = a.taps, rank0 = (h % rep) * nz, p0 = 32 * z, nc = min(32, dv - p0), n_ch = 2 * d + nc;
+    const int tid = threadIdx.x, lane = tid & 31, ns = tid >> 5, n0 = ns * R, p = p0 + lane;
+    const int r = rb.ent_row0[e], slot = rb.ent_slot[e];
+    const bool clustered = rep * nz > 1, low = a.w_a2 != nullptr, live = lane < nc;
+    const int ra4 = (a.a_rank + 3) & ~3, rg4 = (a.g_rank + 3) & ~3;
+    const float* row = a.proj + (size_t)r * a.ld;
+    float* S = a.state + ((size_t)slot * H + h) * d * dv + p;
+    if (clustered) asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");      // (waited for ahead of the first store into another block)
+    float s[R];                                           // the state is requested before anything else
+#pragma unroll
+    for (int i = 0; i < R; ++i) s[i] = (live && n0 + i < d) ? S[(size_t)(n0 + i) * dv] : 0.f;
+    const int dper = (d + nz - 1) / nz, d_lo = min(d, z * dper), nd = min(d, d_lo + dper) - d_lo;      // this block's rows of the decays' product
+    if (low) {                                            // the second factors' rows are on their way to L2 while the convolution runs
+        const int la = (a.a_rank + 63) / 64, lg = (a.g_rank + 63) / 64;
+        for (int i = tid; i < nd * la; i += DS_NT) asm volatile("prefetch.global.L2 [%0];" ::"l"(a.w_a2 + (size_t)(h * d + d_lo + i / la) * a.ld_a2 + 64 * (i % la)));
+        for (int i = tid; i < nc * lg; i += DS_NT) asm volatile("prefetch.global.L2 [%0];" ::"l"(a.w_g2 + (size_t)(h * dv + p0 + i / lg) * a.ld_g2 + 64 * (i % lg)));
+        for (int i = tid; i < ra4; i += DS_NT) xs[i] = i < a.a_rank ? row[a.a_col + i] : 0.f;
+        for (int i = tid; i < rg4; i += DS_NT) xs[ra4 + i] = i < a.g_rank ? row[a.g_col + i] : 0.f;
+    }
+    const float rate = a.rate[h], step_z = row[a.b_col + h], nw = live ? a.norm_w[p] : 0.f;
+    const float dt_b = tid < d ? a.dt_bias[a.per_channel ? h * d + (low ? min(d_lo + tid, d - 1) : tid) : h] : 0.f;
+    float w[DS_CONV][DS_TAPS];                            // convolution: q | k | v channels of this block
+#pragma unroll
+    for (int u = 0; u < DS_CONV; ++u) {
+        const int t = tid + u * DS_NT;
+        if (t >= n_ch) break;
+        const int ch = t < d ? hk * d + t : t < 2 * d ? Hk * d + hk * d + t - d : 2 * Hk * d + h * dv + p0 + t - 2 * d;
+        const float* win = a.conv_state + (size_t)slot * (taps - 1) * C + ch;
+        const float own = row[a.col0 + ch];
+        float acc = 0.f;
+#pragma unroll
+        for (int k = 0; k < DS_TAPS; ++k)
+            if (k < taps) {
+                w[u][k] = k < taps - 1 ? win[(size_t)k * C] : own;
+                acc = fmaf(a.conv_w[(size_t)ch * taps + k], w[u][k], acc);
+            }
+        acc = silu_f(acc);
+        if (t < d) sq[t] = acc; else if (t < 2 * d) sk[t - d] = acc; else sv[t - 2 * d] = acc;
+    }
+    for (int i = d + tid; i < DR; i += DS_NT) { sq[i] = 0.f; sk[i] = 0.f; sdec[i] = 0.f; }
+    __syncthreads();
+    if (low) {
+        constexpr int NR = 4;                             // rows of the second factors in flight per warp
+        for (int i0 = ns * NR; i0 < nd + nc; i0 += DS_NS * NR) {
+            float acc[NR];
+#pragma unroll
+            for (int u = 0; u < NR; ++u) {
+                const int i = min(i0 + u, nd + nc - 1);
+                const bool dec = i < nd;
+                const bf16* wr = dec ? a.w_a2 + (size_t)(h * d + d_lo + i) * a.ld_a2 : a.w_g2 + (size_t)(h * dv + p0 + i - nd) * a.ld_g2;
+                const float* x = dec ? xs : xs + ra4;
+                const int n = dec ? ra4 : rg4;
+                acc[u] = 0.f;
+                for (int k = 4 * lane; k < n; k += 128) {
+                    const uint2 t = *reinterpret_cast<const uint2*>(wr + k);
+                    const float4 xv = *reinterpret_cast<const float4*>(x + k);
+                    acc[u] = fmaf(bf16lo(t.x), xv.x, acc[u]); acc[u] = fmaf(bf16hi(t.x), xv.y, acc[u]);
+                    acc[u] = fmaf(bf16lo(t.y), xv.z, acc[u]); acc[u] = fmaf(bf16hi(t.y), xv.w, acc[u]);
+                }
+            }
+#pragma unroll
+            for (int u = 0; u < NR; ++u) acc[u] = warp_sum(acc[u]);
+            if (lane == 0) {
+#pragma unroll
+                for (int u = 0; u < NR; ++u) if (i0 + u < nd + nc) sz[i0 + u] = acc[u];
+            }
+        }
+    }
+    if (ns == DS_NS - 1) {                                // |q|^2, |k|^2, q . k
+        float qq = 0.f, kk = 0.f, qk = 0.f;
+        for (int i = lane; i < d; i += 32) { qq = fmaf(sq[i], sq[i], qq); kk = fmaf(sk[i], sk[i], kk); qk = fmaf(sq[i], sk[i], qk); }
+        qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
+        if (lane == 0) { scal[0] = a.q_scale / sqrtf(qq + 1e-6f); scal[1] = 1.f / sqrtf(kk + 1e-6f); scal[2] = qk; }
+    }
+    __syncthreads();
+    if (clustered) asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
+    if (low) {
+        if (tid < nd) {
+            const float g = expf(-rate * softplus_f(sz[tid] + dt_b));
+            if (nz > 1) { for (int b = 0; b < nz; ++b) cluster_store(sdec + d_lo + tid, rank0 + b, g); } else sdec[tid] = g;
+        }
+        if (tid < nc) { const float g = sz[nd + tid]; sg[tid] = a.gate_silu ? silu_f(g) : sigmoid_f(g); }
+    } else {
+        if (tid < d) sdec[tid] = expf(-rate * softplus_f(a.z[(size_t)r * a.ldz + (a.per_channel ? h * d + tid : h)] + dt_b));
+        if (tid < nc) { const float g = a.g[(size_t)r * a.ldg + h * dv + p0 + tid]; sg[tid] = a.gate_silu ? silu_f(g) : sigmoid_f(g); }
+    }
+    if (clustered) cluster_sync(); else __syncthreads();  // every block has its decays, and has read the windows
+    const float iq = scal[0], ik = scal[1], qk = scal[2] * iq * ik, beta = sigmoid_f(step_z);
+    float ks = 0.f, qs = 0.f;
+#pragma unroll
+    for (int i = 0; i < R; ++i) { s[i] *= sdec[n0 + i]; ks = fmaf(s[i], sk[n0 + i], ks); qs = fmaf(s[i], sq[n0 + i], qs); }
+    part[0][ns][lane] = ks; part[1][ns][lane] = qs;
+    __syncthreads();
+    float kt = 0.f, qt = 0.f;
+#pragma unroll
+    for (int n = 0; n < DS_NS; ++n) { kt += part[0][n][lane]; qt += part[1][n][lane]; }
+    const float u = live ? beta * (sv[lane] - ik * kt) : 0.f, uk = u * ik, o = live ? fmaf(qk, u, iq * qt) : 0.f;
+    if (ns == 0) {
+        const float ss = warp_sum(o * o);
+        if (lane < nz) { if (nz > 1) cluster_store(ssum + z, rank0 + lane, ss); else ssum[0] = ss; }
+    }
+#pragma unroll
+    for (int i = 0; i < R; ++i) if (live && n0 + i < d) S[(size_t)(n0 + i) * dv] = fmaf(sk[n0 + i], uk, s[i]);
+#pragma unroll
+    for (int v = 0; v < DS_CONV; ++v) {                   // the windows move on; a q / k head's by the first block that shares it
+        const int t = tid + v * DS_NT;
+        if (t >= n_ch) break;
+        if (t < 2 * d && (z || h % rep)) continue;
+        const int ch = t < d ? hk * d + t : t < 2 * d ? Hk * d + hk * d + t - d : 2 * Hk * d + h * dv + p0 + t - 2 * d;
+        float* win = a.conv_state + (size_t)slot * (taps - 1) * C + ch;
+#pragma unroll
+        for (int k = 0; k < DS_TAPS - 1; ++k) if (k < taps - 1) win[(size_t)k * C] = w[v][k + 1];
+    }
+    if (nz > 1) cluster_sync(); else __syncthreads();
+    if (ns == 0 && live) {
+        float tot = 0.f;
+        for (int b = 0; b < nz; ++b) tot += ssum[b];
+        store_act(a.out, r, a.out_col + h * dv + p, o * (a.out_mult / sqrtf(tot / (float)dv + a.eps)) * nw * sg[lane]);
+    }
+}
+
 // ---------------------------------------------------------------------------------------------------------------- the token's own embedding
 __global__ void token_gate_kernel(const float* __restrict__ z, int ldz, int n, const int* __restrict__ ids, const bf16* __restrict__ table, int ldt, int col0, ActOut out) {
     const int r = blockIdx.y, j = blockIdx.x * blockDim.x + threadIdx.x;
@@ -346,6 +490,27 @@ __global__ void __launch_bounds__(128) token_gate_step_kernel(const float* __res
 // ---------------------------------------------------------------------------------------------------------------- launchers
 static bool by_chunks(const DeltaArgs& a) { return a.chunk_ws && a.max_len >= DELTA_CHUNK_MIN; }
 int delta_launch_count(const DeltaArgs& a) { return 3 + (!a.single_rows && a.taps > 1 ? 1 : 0) + (by_chunks(a) ? 1 : 0); }
+bool delta_step_fits(int H, int Hk, int d, int dv, int taps) {
+    return Hk >= 1 && H % Hk == 0 && d >= 1 && d <= 256 && dv >= 1 && (H / Hk) * ((dv + 31) / 32) <= 8 && taps >= 1 && taps <= DS_TAPS;
+}
+int delta_step_launch(cudaStream_t st, const RaggedBatch& rb, const DeltaArgs& a) {
+    if (!delta_step_fits(a.H, a.Hk, a.d, a.dv, a.taps) || rb.T != rb.E || a.a_rank > 4096 || a.g_rank > 4096 || (a.w_a2 && (!a.w_g2 || ((a.ld_a2 | a.ld_g2) & 3)))) return -1000;
+    static_assert(DS_CONV * DS_NT >= 2 * 256 + 32, "a block's channels");
+    const int nz = (a.dv + 31) / 32;
+    const size_t smem = (size_t)(a.a_rank + a.g_rank + 8) * sizeof(float);
+    static SmemOptIn seen[4];
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(a.H * nz, rb.E); cfg.blockDim = dim3(DS_NT); cfg.dynamicSmemBytes = smem; cfg.stream = st;
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = (a.H / a.Hk) * nz; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
+    cfg.attrs = attr; cfg.numAttrs = 1;
+    auto run = [&](auto k, SmemOptIn& s) -> int {
+        if (const int e = ensure_dyn_smem(k, smem, s)) return e;
+        return (int)cudaLaunchKernelEx(&cfg, k, rb, a);
+    };
+    return a.d <= 32 ? run(delta_step_kernel<4>, seen[0]) : a.d <= 64 ? run(delta_step_kernel<8>, seen[1]) : a.d <= 128 ? run(delta_step_kernel<16>, seen[2]) : run(delta_step_kernel<32>, seen[3]);
+}
 int delta_mixer_launch(cudaStream_t st, const RaggedBatch& rb, const DeltaArgs& a) {
     if (a.d < 1 || a.d > 256 || a.dv < 1 || a.Hk < 1 || a.H % a.Hk || a.taps < 1 || !a.conv_w || (a.taps > 1 && !a.conv_state)) return -1000;
     const int units = a.Hk + a.H + (a.per_channel ? a.H : 0) + 1, tile = a.single_rows ? 1 : rb.T >= 1024 ? DP_ROWS : 4, w = std::max(a.d, std::min(a.dv, 128));
