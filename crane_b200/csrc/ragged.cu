@@ -196,7 +196,7 @@ __global__ void attn_prep_kernel(RaggedBatch rb, AttnPrepArgs a) {
         for (int i = threadIdx.x; i < nrot; i += blockDim.x) {
             double sn, cs;
             sincos((double)pos * a.rot_freq[i], &sn, &cs);
-            rot_cs[i] = (float)cs * a.rot_mag; rot_cs[nrot + i] = (float)sn * a.rot_mag;
+            rot_cs[i] = (float)cs; rot_cs[nrot + i] = (float)sn;
         }
         __syncthreads();
     }
@@ -221,46 +221,7 @@ __global__ void attn_prep_kernel(RaggedBatch rb, AttnPrepArgs a) {
     float temp = 1.f;
     if (a.temp_every > 0) temp = 1.f + a.temp_coef * logf((float)((pos + 1) / a.temp_every) + 1.f);
     const int page = a.has_kv ? a.block_table[(size_t)slot * a.max_pages + pos / KV_PAGE] : 0;
-    // value of a projected column: as it is (+ bias), or behind the short convolution over time (a channel belongs to one lane, which
-    // also moves the channel's window on in a step of single rows)
-    const int taps = a.conv_w ? a.conv_taps : 0, conv_ch = (a.H + a.G) * a.d + a.G * a.dv, row_in = r - rb.ent_row0[e];
-    float* win = taps > 1 ? a.conv_state + (size_t)slot * (taps - 1) * conv_ch : nullptr;
-    auto projected = [&](int c) -> float {
-        const float own = row[c];
-        if (!taps) return own + (a.bias ? a.bias[c] : 0.f);
-        const float* w = a.conv_w + (size_t)c * taps;
-        float acc = 0.f;
-        for (int k = 0; k < taps - 1; ++k) {
-            const int back = taps - 1 - k;                // this tap reads the projection `back` tokens ago
-            acc = fmaf(w[k], row_in >= back ? row[c - (ptrdiff_t)back * a.ld] : win[(size_t)(row_in + k) * conv_ch + c], acc);
-        }
-        if (a.single_rows && taps > 1) {
-            for (int k = 1; k < taps - 1; ++k) win[(size_t)(k - 1) * conv_ch + c] = win[(size_t)k * conv_ch + c];
-            win[(size_t)(taps - 2) * conv_ch + c] = own;
-        }
-        return fmaf(w[taps - 1], own, acc);
-    };
     for (int hh = warp; hh < nheads; hh += nw) {
-        if (taps || a.rot_halves) {      // convolved projections and / or the halves-paired rotation: no norm, no temperature
-            const bool isv = hh >= a.H + a.G, isq = hh < a.H;
-            const int width = isv ? a.dv : a.d, half = isv ? 0 : nrot, c0 = isv ? (a.H + a.G) * a.d + (hh - a.H - a.G) * a.dv : hh * a.d;
-            KT* dst = nullptr;
-            if (!isq) {
-                const int g = isv ? hh - a.H - a.G : hh - a.H;
-                dst = (KT*)(isv ? a.v_pool : a.k_pool) + (((size_t)page * a.G + g) * KV_PAGE + (pos % KV_PAGE)) * width;
-            }
-            auto put = [&](int c, float v) {
-                if (isq) store_act(a.q_out, r, c0 + c, v);
-                else kv_store<KT>(dst + c, v, a.kv_lo_off);
-            };
-            for (int i = lane; i < half; i += 32) {
-                const float u = projected(c0 + i), v = projected(c0 + i + half), cs = rot_cs[i], sn = rot_cs[half + i];
-                put(i, u * cs - v * sn);
-                put(i + half, v * cs + u * sn);
-            }
-            for (int c = 2 * half + lane; c < width; c += 32) put(c, projected(c0 + c));
-            continue;
-        }
         if (hh < a.H + nk) {             // q or k head: RMS norm over d (or the row's whole-projection statistic)
             const bool isq = hh < a.H;
             const float* src = row + (size_t)hh * a.d;
@@ -313,6 +274,68 @@ __global__ void attn_prep_kernel(RaggedBatch rb, AttnPrepArgs a) {
                 inv = 1.f / sqrtf(warp_sum(ss) / (float)a.dv + a.eps);
             }
             for (int c = lane; c < a.dv; c += 32) kv_store<KT>(dst + c, (src[c] + (bsrc ? bsrc[c] : 0.f)) * inv, a.kv_lo_off);
+        }
+    }
+}
+
+// The form without a norm whose projections pass a short convolution first and whose rotation pairs dimension i with i + rot_dims / 2.  One
+// warp per (head, tile of rows), the tap window in registers.  The angle is taken in 64-bit and brought into one turn there; its sine
+// and cosine follow in 32-bit.
+constexpr int AC_WARPS = 4;
+template <typename KT, int NC, int TAPS>
+__global__ void __launch_bounds__(AC_WARPS * 32) attn_conv_prep_kernel(RaggedBatch rb, AttnPrepArgs a, int tile) {
+    __shared__ float ys[AC_WARPS][32 * NC];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, hh = blockIdx.y * AC_WARPS + warp, r0 = blockIdx.x * tile, r1 = min(rb.T, r0 + tile);
+    if (hh >= a.H + 2 * a.G) return;
+    const bool isq = hh < a.H, isv = hh >= a.H + a.G;
+    const int width = isv ? a.dv : a.d, g = isv ? hh - a.H - a.G : hh - a.H, c0 = isv ? (a.H + a.G) * a.d + g * a.dv : hh * a.d;
+    const int half = isv ? 0 : a.rot_dims / 2;
+    const ConvSrc cs{a.qkv, a.ld, a.conv_w, a.conv_state, (a.H + a.G) * a.d + a.G * a.dv, a.conv_taps};
+    ConvWalk<NC, TAPS> walk;
+    walk.init(cs, c0, width, lane);
+    double freq[NC];
+#pragma unroll
+    for (int i = 0; i < NC; ++i) { const int c = lane + 32 * i; freq[i] = c < 2 * half ? a.rot_freq[c < half ? c : c - half] : 0.0; }
+    float* yw = ys[warp];
+    for (int rb0 = r0; rb0 < r1; rb0 += 4) {                  // four rows requested before the first is used
+        float x[4][NC];
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+#pragma unroll
+            for (int i = 0; i < NC; ++i) x[u][i] = (rb0 + u < r1 && lane + 32 * i < width) ? a.qkv[(size_t)(rb0 + u) * a.ld + c0 + lane + 32 * i] : 0.f;
+#pragma unroll
+        for (int u = 0; u < 4; ++u) {
+            const int r = rb0 + u;
+            if (r >= r1) break;
+            const int e = rb.row_entry[r], in_entry = r - rb.ent_row0[e], slot = rb.ent_slot[e], pos = rb.row_pos[r];
+            if (r == r0 || in_entry == 0) walk.refill(cs, slot, in_entry, r);
+            float y[NC];
+            walk.step(cs, slot, in_entry, r, x[u], y, a.single_rows != 0 && a.conv_taps > 1);
+            if (half) {                                       // a pair's other half may sit in another lane
+                __syncwarp();
+#pragma unroll
+                for (int i = 0; i < NC; ++i) yw[lane + 32 * i] = y[i];
+                __syncwarp();
+#pragma unroll
+                for (int i = 0; i < NC; ++i) {
+                    const int c = lane + 32 * i;
+                    if (c < 2 * half) {
+                        const double ang = (double)pos * freq[i], turns = rint(ang * 0.15915494309189535);
+                        float sn, cn;
+                        sincosf((float)(ang - turns * 6.283185307179586), &sn, &cn);
+                        y[i] = a.rot_mag * (c < half ? y[i] * cn - yw[c + half] * sn : y[i] * cn + yw[c - half] * sn);
+                    }
+                }
+            }
+            if (isq) {
+#pragma unroll
+                for (int i = 0; i < NC; ++i) if (lane + 32 * i < width) store_act(a.q_out, r, c0 + lane + 32 * i, y[i]);
+            } else {
+                const int page = a.block_table[(size_t)slot * a.max_pages + pos / KV_PAGE];
+                KT* dst = (KT*)(isv ? a.v_pool : a.k_pool) + (((size_t)page * a.G + g) * KV_PAGE + (pos % KV_PAGE)) * width;
+#pragma unroll
+                for (int i = 0; i < NC; ++i) if (lane + 32 * i < width) kv_store<KT>(dst + lane + 32 * i, y[i], a.kv_lo_off);
+            }
         }
     }
 }
@@ -1187,11 +1210,25 @@ int silu_glu_launch(cudaStream_t st, const float* gu, int ld, int T, int F, cons
     silu_glu_kernel<<<dim3((F + 127) / 128, T), 128, 0, st>>>(gu, ld, F, out, limit, bias);
     return last_err();
 }
+template <typename KT>
+static int attn_conv_prep_launch(cudaStream_t st, const RaggedBatch& rb, const AttnPrepArgs& a) {
+    const int w = std::max(a.d, a.dv), units = a.H + 2 * a.G, tile = a.single_rows ? 1 : rb.T >= 1024 ? 16 : 4;
+    if (w > 256 || a.conv_taps < 1 || (a.conv_taps > 1 && !a.conv_state) || !a.no_norm || !a.has_kv || a.v_from_k || a.v_unit || a.bias || a.q_head_scale) return -1000;
+    const dim3 grid((rb.T + tile - 1) / tile, (units + AC_WARPS - 1) / AC_WARPS);
+    auto run = [&](auto k0, auto k1, auto k2, auto k3, auto k4) {
+        auto k = a.conv_taps == 1 ? k1 : a.conv_taps == 2 ? k2 : a.conv_taps == 3 ? k3 : a.conv_taps == 4 ? k4 : k0;
+        k<<<grid, AC_WARPS * 32, 0, st>>>(rb, a, tile);
+    };
+    if (w <= 64) run(attn_conv_prep_kernel<KT, 2, 0>, attn_conv_prep_kernel<KT, 2, 1>, attn_conv_prep_kernel<KT, 2, 2>, attn_conv_prep_kernel<KT, 2, 3>, attn_conv_prep_kernel<KT, 2, 4>);
+    else if (w <= 128) run(attn_conv_prep_kernel<KT, 4, 0>, attn_conv_prep_kernel<KT, 4, 1>, attn_conv_prep_kernel<KT, 4, 2>, attn_conv_prep_kernel<KT, 4, 3>, attn_conv_prep_kernel<KT, 4, 4>);
+    else run(attn_conv_prep_kernel<KT, 8, 0>, attn_conv_prep_kernel<KT, 8, 1>, attn_conv_prep_kernel<KT, 8, 2>, attn_conv_prep_kernel<KT, 8, 3>, attn_conv_prep_kernel<KT, 8, 4>);
+    return last_err();
+}
 int attn_prep_launch(cudaStream_t st, const RaggedBatch& rb, const AttnPrepArgs& a) {
     if (a.rot_dims < 0 || (a.rot_dims & 1) || a.rot_dims > a.d || a.rot_dims > 4096) return -1000;
     if (a.v_from_k && a.d != a.dv) return -1000;
-    if ((a.conv_w || a.rot_halves) && (!a.no_norm || !a.has_kv || a.v_from_k || a.v_unit || a.bias || a.q_head_scale)) return -1000;
-    if (a.conv_w && (a.conv_taps < 1 || (a.conv_taps > 1 && !a.conv_state))) return -1000;
+    if (a.rot_halves != (a.conv_w ? 1 : 0) || (a.rot_mag != 1.f && !a.conv_w)) return -1000;
+    if (a.conv_w) return a.kv_f32 ? attn_conv_prep_launch<float>(st, rb, a) : attn_conv_prep_launch<bf16>(st, rb, a);
     const size_t sm = (size_t)a.rot_dims * sizeof(float);
     if (a.kv_f32) attn_prep_kernel<float><<<rb.T, 256, sm, st>>>(rb, a);
     else attn_prep_kernel<bf16><<<rb.T, 256, sm, st>>>(rb, a);

@@ -91,9 +91,10 @@ struct AttnPrepArgs {
     int v_unit = 0;                   // 1: every value head is divided by its root mean square over dv (eps, no weight) before it is cached
     int v_from_k = 0;                 // 1: the row has no value columns; the cached value of a head is its key as projected (+ bias), before the norm (dv == d)
     const float* q_head_scale = nullptr;   // nullable [H]: head h's normalised query is multiplied by q_head_scale[h]
-    int rot_halves = 0;               // 1: dimension i turns together with dimension i + rot_dims / 2 (instead of pairs (2i, 2i + 1))
+    // The form with a short convolution (conv_w != nullptr; no norm, no temperature, no bias; d and dv <= 256):
+    int rot_halves = 0;               // 1, with conv_w only: dimension i turns together with dimension i + rot_dims / 2 (instead of pairs (2i, 2i + 1))
     float rot_mag = 1.f;              // factor on the rotation's cosines and sines
-    // a short causal convolution over time on every projected channel (q | k | v columns), ahead of everything else:
+    // a causal convolution over time on every projected channel (q | k | v columns), ahead of everything else:
     // u_t = sum_j conv_w[c, j] * p_(t - taps + 1 + j), p the projections; inputs ahead of the entry come from the carried window
     const float* conv_w = nullptr;    // [(H + G) * d + G * dv, taps]
     int conv_taps = 0;

@@ -21,80 +21,17 @@ __device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
 
 // ---------------------------------------------------------------------------------------------------------------- prep
-// Walks rows r0 .. r1 - 1 of NC * 32 channels starting at column c0 (lane owns c0 + lane + 32 i, i < NC, below c0 + width): emit(r, y) gets
-// the convolved values of row r.  TAPS > 0: the tap window lives in registers; TAPS == 0: any number of taps, read back from memory.
-template <int NC, int TAPS>
-struct ConvWalk {
-    float w[NC][TAPS > 0 ? TAPS : 1], h[NC][TAPS > 1 ? TAPS - 1 : 1];
-    int c0, width, lane, C;
-    __device__ __forceinline__ void init(const DeltaArgs& a, int c0_, int width_, int lane_) {
-        c0 = c0_; width = width_; lane = lane_; C = 2 * a.Hk * a.d + a.H * a.dv;
-        if constexpr (TAPS > 0) {
-#pragma unroll
-            for (int i = 0; i < NC; ++i) {
-                const int c = lane + 32 * i;
-#pragma unroll
-                for (int k = 0; k < TAPS; ++k) w[i][k] = c < width ? a.conv_w[(size_t)(c0 + c) * TAPS + k] : 0.f;
-            }
-        }
-    }
-    __device__ __forceinline__ float before(const DeltaArgs& a, int slot, int in_entry, int r, int c, int k) const {      // what tap k of row r reads
-        const int back = a.taps - 1 - k;
-        return in_entry >= back ? a.proj[(size_t)(r - back) * a.ld + a.col0 + c0 + c] : a.conv_state[((size_t)slot * (a.taps - 1) + in_entry + k) * C + c0 + c];
-    }
-    __device__ __forceinline__ void refill(const DeltaArgs& a, int slot, int in_entry, int r) {
-        if constexpr (TAPS > 1) {
-#pragma unroll
-            for (int i = 0; i < NC; ++i) {
-                const int c = lane + 32 * i;
-#pragma unroll
-                for (int k = 0; k < TAPS - 1; ++k) h[i][k] = c < width ? before(a, slot, in_entry, r, c, k) : 0.f;
-            }
-        }
-    }
-    // y[i] of row r from its own inputs x[i]; with `move` the carried window of the row's sequence moves on
-    __device__ __forceinline__ void step(const DeltaArgs& a, int slot, int in_entry, int r, const float* x, float* y, bool move) {
-#pragma unroll
-        for (int i = 0; i < NC; ++i) {
-            const int c = lane + 32 * i;
-            float acc = 0.f;
-            if constexpr (TAPS > 0) {
-#pragma unroll
-                for (int k = 0; k < TAPS - 1; ++k) acc = fmaf(w[i][k], h[i][k], acc);
-                acc = fmaf(w[i][TAPS - 1], x[i], acc);
-                if (TAPS > 1) {
-#pragma unroll
-                    for (int k = 0; k < TAPS - 2; ++k) h[i][k] = h[i][k + 1];
-                    h[i][TAPS - 2] = x[i];
-                    if (move && c < width) {
-#pragma unroll
-                        for (int k = 0; k < TAPS - 1; ++k) a.conv_state[((size_t)slot * (TAPS - 1) + k) * C + c0 + c] = h[i][k];
-                    }
-                }
-            } else if (c < width) {
-                for (int k = 0; k < a.taps - 1; ++k) acc = fmaf(a.conv_w[(size_t)(c0 + c) * a.taps + k], before(a, slot, in_entry, r, c, k), acc);
-                acc = fmaf(a.conv_w[(size_t)(c0 + c) * a.taps + a.taps - 1], x[i], acc);
-                if (move) {
-                    float* win = a.conv_state + (size_t)slot * (a.taps - 1) * C + c0 + c;
-                    for (int k = 1; k < a.taps - 1; ++k) win[(size_t)(k - 1) * C] = win[(size_t)k * C];
-                    win[(size_t)(a.taps - 2) * C] = x[i];
-                }
-            }
-            y[i] = acc;
-        }
-    }
-};
-
 constexpr int DP_ROWS = 16;      // rows a warp walks
 template <int NC, int TAPS>
 __global__ void __launch_bounds__(128) delta_prep_kernel(RaggedBatch rb, DeltaArgs a, int tile) {
     const int lane = threadIdx.x & 31, unit = blockIdx.y * 4 + (threadIdx.x >> 5), r0 = blockIdx.x * tile, r1 = min(rb.T, r0 + tile);
     const int Hk = a.Hk, H = a.H, d = a.d, dv = a.dv, n_dec = a.per_channel ? H : 0;
     if (unit >= Hk + H + n_dec + 1) return;
+    const ConvSrc cs{a.proj + a.col0, a.ld, a.conv_w, a.conv_state, 2 * Hk * d + H * dv, a.taps};
     if (unit < Hk) {                                          // a q / k head: convolution, SiLU, unit vectors, their product
         ConvWalk<NC, TAPS> q, k;
-        q.init(a, unit * d, d, lane);
-        k.init(a, (Hk + unit) * d, d, lane);
+        q.init(cs, unit * d, d, lane);
+        k.init(cs, (Hk + unit) * d, d, lane);
         for (int rb0 = r0; rb0 < r1; rb0 += 4) {              // four rows requested before the first is used
             float xq[4][NC], xk[4][NC];
 #pragma unroll
@@ -110,10 +47,10 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(RaggedBatch rb, DeltaAr
                 const int r = rb0 + u;
                 if (r >= r1) break;
                 const int e = rb.row_entry[r], in_entry = r - rb.ent_row0[e], slot = rb.ent_slot[e];
-                if (r == r0 || in_entry == 0) { q.refill(a, slot, in_entry, r); k.refill(a, slot, in_entry, r); }
+                if (r == r0 || in_entry == 0) { q.refill(cs, slot, in_entry, r); k.refill(cs, slot, in_entry, r); }
                 float yq[NC], yk[NC], sq = 0.f, sk = 0.f, sqk = 0.f;
-                q.step(a, slot, in_entry, r, xq[u], yq, a.single_rows != 0 && a.taps > 1);
-                k.step(a, slot, in_entry, r, xk[u], yk, a.single_rows != 0 && a.taps > 1);
+                q.step(cs, slot, in_entry, r, xq[u], yq, a.single_rows != 0 && a.taps > 1);
+                k.step(cs, slot, in_entry, r, xk[u], yk, a.single_rows != 0 && a.taps > 1);
 #pragma unroll
                 for (int i = 0; i < NC; ++i) {
                     yq[i] = silu_f(yq[i]); yk[i] = silu_f(yk[i]);
@@ -134,7 +71,7 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(RaggedBatch rb, DeltaAr
         const int h = unit - Hk;
         for (int cb = 0; cb < dv; cb += 32 * NC) {
             ConvWalk<NC, TAPS> v;
-            v.init(a, 2 * Hk * d + h * dv + cb, min(32 * NC, dv - cb), lane);
+            v.init(cs, 2 * Hk * d + h * dv + cb, min(32 * NC, dv - cb), lane);
             for (int rb0 = r0; rb0 < r1; rb0 += 4) {
                 float x[4][NC];
 #pragma unroll
@@ -147,9 +84,9 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(RaggedBatch rb, DeltaAr
                     const int r = rb0 + u;
                     if (r >= r1) break;
                     const int e = rb.row_entry[r], in_entry = r - rb.ent_row0[e], slot = rb.ent_slot[e];
-                    if (r == r0 || in_entry == 0) v.refill(a, slot, in_entry, r);
+                    if (r == r0 || in_entry == 0) v.refill(cs, slot, in_entry, r);
                     float y[NC];
-                    v.step(a, slot, in_entry, r, x[u], y, a.single_rows != 0 && a.taps > 1);
+                    v.step(cs, slot, in_entry, r, x[u], y, a.single_rows != 0 && a.taps > 1);
 #pragma unroll
                     for (int i = 0; i < NC; ++i) if (lane + 32 * i < v.width) a.v[((size_t)r * H + h) * dv + cb + lane + 32 * i] = silu_f(y[i]);
                 }

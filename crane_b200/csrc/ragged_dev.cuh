@@ -24,6 +24,76 @@ __device__ __forceinline__ void cp_async4(void* smem_dst, const void* gsrc) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_u32(smem_dst)), "l"(gsrc) : "memory");
 }
 
+// A short causal convolution over time that a warp walks row by row: NC * 32 channels starting at c0 (a lane owns c0 + lane + 32 i, i < NC,
+// below c0 + width).  TAPS > 0: the tap window lives in registers; TAPS == 0: any number of taps, read back from memory.
+struct ConvSrc {
+    const float* in; int ld;          // [T, ld]
+    const float* w;                   // [C, taps], last column on the current token
+    float* state;                     // [slots, taps - 1, C] the inputs ahead of the step's rows
+    int C, taps;
+};
+template <int NC, int TAPS>
+struct ConvWalk {
+    float w[NC][TAPS > 0 ? TAPS : 1], h[NC][TAPS > 1 ? TAPS - 1 : 1];
+    int c0, width, lane, C;
+    __device__ __forceinline__ void init(const ConvSrc& a, int c0_, int width_, int lane_) {
+        c0 = c0_; width = width_; lane = lane_; C = a.C;
+        if constexpr (TAPS > 0) {
+#pragma unroll
+            for (int i = 0; i < NC; ++i) {
+                const int c = lane + 32 * i;
+#pragma unroll
+                for (int k = 0; k < TAPS; ++k) w[i][k] = c < width ? a.w[(size_t)(c0 + c) * TAPS + k] : 0.f;
+            }
+        }
+    }
+    __device__ __forceinline__ float before(const ConvSrc& a, int slot, int in_entry, int r, int c, int k) const {      // what tap k of row r reads
+        const int back = a.taps - 1 - k;
+        return in_entry >= back ? a.in[(size_t)(r - back) * a.ld + c0 + c] : a.state[((size_t)slot * (a.taps - 1) + in_entry + k) * C + c0 + c];
+    }
+    __device__ __forceinline__ void refill(const ConvSrc& a, int slot, int in_entry, int r) {
+        if constexpr (TAPS > 1) {
+#pragma unroll
+            for (int i = 0; i < NC; ++i) {
+                const int c = lane + 32 * i;
+#pragma unroll
+                for (int k = 0; k < TAPS - 1; ++k) h[i][k] = c < width ? before(a, slot, in_entry, r, c, k) : 0.f;
+            }
+        }
+    }
+    // y[i] of row r from its own inputs x[i]; with `move` the carried window of the row's sequence moves on
+    __device__ __forceinline__ void step(const ConvSrc& a, int slot, int in_entry, int r, const float* x, float* y, bool move) {
+#pragma unroll
+        for (int i = 0; i < NC; ++i) {
+            const int c = lane + 32 * i;
+            float acc = 0.f;
+            if constexpr (TAPS > 0) {
+#pragma unroll
+                for (int k = 0; k < TAPS - 1; ++k) acc = fmaf(w[i][k], h[i][k], acc);
+                acc = fmaf(w[i][TAPS - 1], x[i], acc);
+                if (TAPS > 1) {
+#pragma unroll
+                    for (int k = 0; k < TAPS - 2; ++k) h[i][k] = h[i][k + 1];
+                    h[i][TAPS - 2] = x[i];
+                    if (move && c < width) {
+#pragma unroll
+                        for (int k = 0; k < TAPS - 1; ++k) a.state[((size_t)slot * (TAPS - 1) + k) * C + c0 + c] = h[i][k];
+                    }
+                }
+            } else if (c < width) {
+                for (int k = 0; k < a.taps - 1; ++k) acc = fmaf(a.w[(size_t)(c0 + c) * a.taps + k], before(a, slot, in_entry, r, c, k), acc);
+                acc = fmaf(a.w[(size_t)(c0 + c) * a.taps + a.taps - 1], x[i], acc);
+                if (move) {
+                    float* win = a.state + (size_t)slot * (a.taps - 1) * C + c0 + c;
+                    for (int k = 1; k < a.taps - 1; ++k) win[(size_t)(k - 1) * C] = win[(size_t)k * C];
+                    win[(size_t)(a.taps - 2) * C] = x[i];
+                }
+            }
+            y[i] = acc;
+        }
+    }
+};
+
 // KV page elements: f32, or bf16 with an optional low-order plane `lo` elements further on (x ~= hi + lo, ~16 mantissa bits)
 template <typename KT> __device__ __forceinline__ float kv_load(const KT* p, long long lo);
 template <> __device__ __forceinline__ float kv_load<float>(const float* p, long long) { return *p; }
