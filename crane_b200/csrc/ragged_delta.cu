@@ -97,8 +97,13 @@ __global__ void __launch_bounds__(128) delta_prep_kernel(RaggedBatch rb, DeltaAr
         const float rate = a.rate[h];
         for (int c = lane; c < d; c += 32) {
             const float b = a.dt_bias[h * d + c];
-#pragma unroll 4
-            for (int r = r0; r < r1; ++r) a.dec[(size_t)r * a.lddec + h * d + c] = expf(-rate * softplus_f(a.z[(size_t)r * a.ldz + h * d + c] + b));
+            for (int rb0 = r0; rb0 < r1; rb0 += 8) {          // (dec may be z itself: the rows are requested ahead of the first store)
+                float z[8];
+#pragma unroll
+                for (int u = 0; u < 8; ++u) z[u] = rb0 + u < r1 ? a.z[(size_t)(rb0 + u) * a.ldz + h * d + c] : 0.f;
+#pragma unroll
+                for (int u = 0; u < 8; ++u) if (rb0 + u < r1) a.dec[(size_t)(rb0 + u) * a.lddec + h * d + c] = expf(-rate * softplus_f(z[u] + b));
+            }
         }
     } else {                                                  // step sizes (and the decays of whole heads)
         for (int i = lane; i < (r1 - r0) * H; i += 32) {
