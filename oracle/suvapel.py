@@ -112,12 +112,12 @@ def attend(q, k, v, q_pos, scale, mask):
     """Softmax attention of rows q [S, H, d] at positions q_pos over the keys k [n, G, d] / values v [n, G, dv]."""
     S, H, _ = q.shape
     G, dv = v.shape[1], v.shape[2]
+    group = torch.arange(H) // (H // G)          # key / value head of every query head
     out = torch.zeros(S, H, dv, dtype=q.dtype)
     for i in range(S):
         js = visible(int(q_pos[i]), mask)
-        for h in range(H):
-            g = h // (H // G)
-            out[i, h] = torch.softmax((k[js, g] @ q[i, h]) * scale, 0) @ v[js, g]
+        p = torch.softmax((k[js][:, group] * q[i]).sum(-1) * scale, 0)          # [keys, H]
+        out[i] = (p[:, :, None] * v[js][:, group]).sum(0)
     return out
 
 
