@@ -1,9 +1,11 @@
 // The gated delta rule on ragged batches (see ragged.cuh), and the embedding of the token that joins behind a layer.
 //   prep : per (q / k head | value head | gates): convolution over time with the carried window, SiLU, unit norms, q . k, the decays
 //          and step sizes -- f32 throughout, one warp per head and tile of rows, the tap window in registers;
-//   scan : the recurrence token by token (long portions: 16 tokens at a time, ragged_delta_chunk.cu), a thread keeps its share of the state in registers for the whole portion, the inputs of
-//          DR_CH tokens at a time staged in shared memory (cp.async, double-buffered);
-//   out  : norm over the value width, gate.
+//   scan : the recurrence token by token, a thread keeps its share of the state in registers for the whole portion, the inputs of DR_CH
+//          tokens at a time staged in shared memory (cp.async, double-buffered); long portions go 16 tokens at a time instead
+//          (ragged_delta_chunk.cu);
+//   out  : norm over the value width, gate;
+//   step : all of it in one launch, for steps whose entries are one row each.
 // A row's result depends on its own sequence only: the split of the state over lanes and the order of the lane sums are launch
 // constants.
 #include "ragged.cuh"
