@@ -661,6 +661,14 @@ class SuvapelModel(FosovikModel):
     channel.  Same entry points and engine options as `FosovikModel`."""
 
 
+class RupulixModel(FosovikModel):
+    """A layer-list decoder ("architecture": "Rupulix"): the residual is several parallel streams; every sublayer reads the RMS norm of
+    their weighted sum and writes back through a mixing table.  Mixers: sliding-window latent attention with a rotated part beside the
+    latent one and a learned sink, or attention whose heads' scores are mixed ahead of the softmax beside a gated linear recurrence
+    (real decays, short convolution, f32 state); feed-forward: squared ReLU.  A span of the layer list may repeat with pages and states
+    of its own per pass; the head is the embedding table.  Same entry points and engine options as `FosovikModel`."""
+
+
 # config.json -> model class, as `model_factory::create_backend` picks a backend by architecture (crane-serve/src/engine/model_factory.rs:471-560)
 def model_class(config: dict):
     if config.get("architecture") == "Fosovik":
@@ -673,6 +681,8 @@ def model_class(config: dict):
         return PuzonexModel
     if config.get("architecture") == "Suvapel":
         return SuvapelModel
+    if config.get("architecture") == "Rupulix":
+        return RupulixModel
     if "talker_config" in config:
         return Qwen3TTSModel
     if "vision_config" in config:

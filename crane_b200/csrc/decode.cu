@@ -218,7 +218,8 @@ gemv_kernel(GemvArgs a) {
                     if (a.out_scale) add *= a.out_scale[r0 + i];
                     if (a.gate) add *= 1.f / (1.f + expf(-(a.gate[(size_t)b * a.ldg + r0 + i] + (a.gate_bias ? a.gate_bias[r0 + i] : 0.f))));
                     *yp += add;
-                } else *yp = v;
+                } else if constexpr (EPI == GEMV_RELU2) { const float p = fmaxf(v, 0.f); *yp = p * p; }
+                else *yp = v;
                 if constexpr (EPI == GEMV_LOGITS_ARGMAX) {
                     if (v > bestv[b]) { bestv[b] = v; besti[b] = r0 + i; }   // a thread's rows ascend: first maximum wins
                 }
@@ -334,6 +335,7 @@ static int gemv_launch_b(cudaStream_t st, int epi, bool norm, const GemvArgs& a,
         case GEMV_STORE:
             return norm ? gemv_launch_t<B, GEMV_STORE, true>(st, a, num_sms, pdl) : gemv_launch_t<B, GEMV_STORE, false>(st, a, num_sms, pdl);
         case GEMV_RESID: return gemv_launch_t<B, GEMV_RESID, false>(st, a, num_sms, pdl);
+        case GEMV_RELU2: return norm ? -1000 : gemv_launch_t<B, GEMV_RELU2, false>(st, a, num_sms, pdl);
         case GEMV_SILU_MUL:
             return norm ? gemv_launch_t<B, GEMV_SILU_MUL, true>(st, a, num_sms, pdl) : gemv_launch_t<B, GEMV_SILU_MUL, false>(st, a, num_sms, pdl);
         case GEMV_LOGITS_ARGMAX: return gemv_launch_t<B, GEMV_LOGITS_ARGMAX, true>(st, a, num_sms, pdl);

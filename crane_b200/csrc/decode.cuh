@@ -31,7 +31,7 @@ struct SeqState {
     int pad;
 };
 
-enum GemvEpi : int { GEMV_STORE = 0, GEMV_RESID = 1, GEMV_SILU_MUL = 2, GEMV_LOGITS_ARGMAX = 3 };
+enum GemvEpi : int { GEMV_STORE = 0, GEMV_RESID = 1, GEMV_SILU_MUL = 2, GEMV_LOGITS_ARGMAX = 3, GEMV_RELU2 = 4 };      // GEMV_RELU2: y = max(W x, 0)^2
 
 struct GemvArgs {
     const bf16* W;          // [N, K] row-major (gate/up rows interleaved for GEMV_SILU_MUL)

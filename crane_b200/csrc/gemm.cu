@@ -116,6 +116,7 @@ __device__ __forceinline__ void epi_store32(const GemmEpi& ep, int m, int n, flo
                 float a = v[j + 2 * t], b = v[j + 2 * t + 1];
                 if constexpr (MODE == EPI_GELU_ERF_BF16) { a = gelu_erf_f(a); b = gelu_erf_f(b); }
                 else if constexpr (MODE == EPI_GELU_TANH_BF16) { a = gelu_tanh_f(a); b = gelu_tanh_f(b); }
+                else if constexpr (MODE == EPI_RELU2_BF16) { a = fmaxf(a, 0.f); b = fmaxf(b, 0.f); a *= a; b *= b; }
                 split_bf16x2(a, b, p[t], q[t]);
             }
             *reinterpret_cast<uint4*>(o + j) = make_uint4(p[0], p[1], p[2], p[3]);
@@ -685,6 +686,7 @@ int gemm_bf16_launch(cudaStream_t stream, const bf16* A, const bf16* A_lo, int l
         case EPI_SILU_MUL_BF16:  return launch_mode<EPI_SILU_MUL_BF16>(stream, A, A_lo, lda, W, M, N, K, epi, use_simt);
         case EPI_GELU_ERF_BF16:  return launch_mode<EPI_GELU_ERF_BF16>(stream, A, A_lo, lda, W, M, N, K, epi, use_simt);
         case EPI_GELU_TANH_BF16: return launch_mode<EPI_GELU_TANH_BF16>(stream, A, A_lo, lda, W, M, N, K, epi, use_simt);
+        case EPI_RELU2_BF16:     return launch_mode<EPI_RELU2_BF16>(stream, A, A_lo, lda, W, M, N, K, epi, use_simt);
         default: return -1000;
     }
 }

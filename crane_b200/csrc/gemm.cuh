@@ -23,7 +23,8 @@ enum GemmEpiMode : int {
     EPI_SILU_MUL_BF16 = 3, // W rows interleaved (gate_j, up_j): out bf16 [M, ldo][j] = silu(acc[2j]) * acc[2j+1]; with GemmEpi::glu_limit > 0
                            // the clamped unit instead: g = min(acc[2j], L), u = clamp(acc[2j+1], -L, L), out = g * sigmoid(1.702 g) * (u + 1)
     EPI_GELU_ERF_BF16 = 4, // out bf16 = gelu_erf(acc + bias)
-    EPI_GELU_TANH_BF16 = 5 // out bf16 = gelu_tanh(acc + bias)
+    EPI_GELU_TANH_BF16 = 5, // out bf16 = gelu_tanh(acc + bias)
+    EPI_RELU2_BF16 = 6     // out bf16 = max(acc + bias, 0)^2
 };
 
 struct GemmEpi {

@@ -68,6 +68,10 @@ struct FlashArgs {
     int keep_first = 0;                 // window > 0: the first keep_first keys of the sequence stay visible behind the window
     int gate_heads = 0;                 // 1: gate holds one number per head ([rows, g_stride], head h at h)
     float out_mult = 1.f;               // factor on every output
+    // flash_ragged_launch: widths that are not the kernel's own.  A query head / a cached key is a row of k_w columns, a cached value one of v_w
+    // (multiples of 8, zeros or anything finite against zeros behind the real width), a head's output dv columns (even)
+    int k_w = 0, v_w = 0, dv = 0;
+    int k_heads = 0;                    // key heads in k_pool (0: nkv): head h reads key head h / (nh / k_heads) and value head h / (nh / nkv)
 };
 
 // quantised KV pages <-> the bf16 (hi + lo) scratch the prefill kernels read and write (see prefill.cu)
@@ -90,6 +94,9 @@ int rope_append_launch(cudaStream_t st, int D, const RopeAppendArgs& a);
 // D: key width; DV: value width (0: equal).  Widths that differ: paged causal launches with (64, 128) or (128, 64); flash_widths_fit tells.
 int flash_prefill_launch(cudaStream_t st, int D, bool causal, bool paged, const FlashArgs& a, int DV = 0);
 inline bool flash_widths_fit(int D, int DV) { return (D == DV && (D == 64 || D == 128 || D == 256)) || (D == 64 && DV == 128) || (D == 128 && DV == 64); }
+// Ragged causal launches over paged caches with any widths (FlashArgs::k_w, v_w, dv): the tile is the next larger one the kernel is compiled for.
+int flash_ragged_launch(cudaStream_t st, const FlashArgs& a);
+inline bool flash_ragged_fits(int k_w, int v_w, int dv) { return k_w > 0 && k_w <= 256 && (k_w & 7) == 0 && v_w >= dv && v_w <= 256 && (v_w & 7) == 0 && dv > 0 && (dv & 1) == 0; }
 int gate_mul_launch(cudaStream_t st, bf16* attn, const float* qkv, int S, int nh, int D, int q_stride, int row_width, long long lo_off = 0);
 int set_rows_launch(cudaStream_t st, float* x, int H, const int* rows, int n, const float* src, bool add);
 int cast_f32_bf16_launch(cudaStream_t st, const float* src, bf16* dst, size_t n, long long lo_off = 0);

@@ -173,6 +173,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict
                 if (MODE == LIN_RESID && bias) v += bias[n];
                 if (MODE == LIN_RESID && col_scale) v *= col_scale[n];
                 if (MODE == LIN_RESID && gate) v *= 1.f / (1.f + expf(-(gate[(size_t)m * ldg + n] + (gate_bias ? gate_bias[n] : 0.f))));
+                if (MODE == LIN_RELU2) { v = fmaxf(v, 0.f); v *= v; }
                 *p = (MODE == LIN_RESID) ? *p + v : v;
             }
         }
@@ -180,12 +181,14 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict
 
 // ---------------------------------------------------------------------------------------------------------------- attention
 // One warp per (row, head): q -> rms_norm(q) [* w] * temp(pos), rotated; k -> rms_norm(k) [* w], rotated, into its page; v into its page.
-// The rotation turns neighbouring pairs (2i, 2i + 1) of the first rot_dims dimensions by pos * rot_freq[i]; the row's cosines and
-// sines are taken once per row, in 64-bit, and shared by its heads.
+// The rotation turns pairs of the first rot_dims dimensions -- neighbours (2i, 2i + 1), or (i, i + rot_dims / 2) -- by pos * rot_freq[i]; the
+// row's cosines and sines are taken once per row, in 64-bit, and shared by its heads.  With `talk` the row's prepared queries meet in
+// shared memory and leave as the mixed ones.
 template <typename KT>
 __global__ void attn_prep_kernel(RaggedBatch rb, AttnPrepArgs a) {
-    extern __shared__ float rot_cs[];                    // [rot_dims / 2] cos, then sin
+    extern __shared__ float rot_cs[];                    // [rot_dims / 2] cos, then sin; with `talk` [H * d] queries behind them
     __shared__ float whole[2][8];
+    float* sq = rot_cs + a.rot_dims;
     const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
     const int e = rb.row_entry[r], pos = rb.row_pos[r], slot = rb.ent_slot[e];
     const float* row = a.qkv + (size_t)r * a.ld;
@@ -236,29 +239,32 @@ __global__ void attn_prep_kernel(RaggedBatch rb, AttnPrepArgs a) {
             KT* dst = nullptr; KT* dstv = nullptr;
             if (!isq) {
                 const size_t at = ((size_t)page * a.G + (hh - a.H)) * KV_PAGE + (pos % KV_PAGE);
-                dst = (KT*)a.k_pool + at * a.d;
+                dst = a.talk ? (KT*)a.k_pool + ((size_t)page * KV_PAGE + pos % KV_PAGE) * a.k_row + (size_t)(hh - a.H) * a.d : (KT*)a.k_pool + at * a.d;
                 if (a.v_from_k) dstv = (KT*)a.v_pool + at * a.dv;
             }
-            // a lane owns the pairs (2i, 2i + 1), i = lane, lane + 32, ...: both halves of a rotated pair are in one thread
-            for (int c = 2 * lane; c < a.d; c += 64) {
-                const float u0 = src[c] + (bsrc ? bsrc[c] : 0.f), v0 = (c + 1 < a.d) ? src[c + 1] + (bsrc ? bsrc[c + 1] : 0.f) : 0.f;
+            // a lane owns the pairs i = lane, lane + 32, ...: both halves of a rotated pair are in one thread
+            for (int i = lane; 2 * i < a.d; i += 32) {
+                const bool halves = a.rot_halves && i < nrot;
+                const int c = halves ? i : 2 * i, c1 = halves ? i + nrot : c + 1;
+                const float u0 = src[c] + (bsrc ? bsrc[c] : 0.f), v0 = (c1 < a.d) ? src[c1] + (bsrc ? bsrc[c1] : 0.f) : 0.f;
                 if (dstv) {               // the value is the key as projected
                     kv_store<KT>(dstv + c, u0, a.kv_lo_off);
-                    if (c + 1 < a.d) kv_store<KT>(dstv + c + 1, v0, a.kv_lo_off);
+                    if (c1 < a.d) kv_store<KT>(dstv + c1, v0, a.kv_lo_off);
                 }
                 float u = u0 * inv, v = v0 * inv;
-                if (nwt) { u *= nwt[c]; if (c + 1 < a.d) v *= nwt[c + 1]; }
-                if (c + 1 < a.rot_dims) {
-                    const float cs = rot_cs[c >> 1], sn = rot_cs[nrot + (c >> 1)];
+                if (nwt) { u *= nwt[c]; if (c1 < a.d) v *= nwt[c1]; }
+                if (i < nrot) {
+                    const float cs = rot_cs[i], sn = rot_cs[nrot + i];
                     const float u2 = u * cs - v * sn, v2 = v * cs + u * sn;
                     u = u2; v = v2;
                 }
-                if (isq) {
+                if (isq && a.talk) { sq[hh * a.d + c] = u; if (c1 < a.d) sq[hh * a.d + c1] = v; }
+                else if (isq) {
                     store_act(a.q_out, r, hh * a.d + c, u);
-                    if (c + 1 < a.d) store_act(a.q_out, r, hh * a.d + c + 1, v);
+                    if (c1 < a.d) store_act(a.q_out, r, hh * a.d + c1, v);
                 } else {
                     kv_store<KT>(dst + c, u, a.kv_lo_off);
-                    if (c + 1 < a.d) kv_store<KT>(dst + c + 1, v, a.kv_lo_off);
+                    if (c1 < a.d) kv_store<KT>(dst + c1, v, a.kv_lo_off);
                 }
             }
         } else {
@@ -266,7 +272,7 @@ __global__ void attn_prep_kernel(RaggedBatch rb, AttnPrepArgs a) {
             const size_t off = (size_t)(a.H + a.G) * a.d + (size_t)g * a.dv;
             const float* src = row + off;
             const float* bsrc = a.bias ? a.bias + off : nullptr;
-            KT* dst = (KT*)a.v_pool + (((size_t)page * a.G + g) * KV_PAGE + (pos % KV_PAGE)) * a.dv;
+            KT* dst = (KT*)a.v_pool + (((size_t)page * a.G + g) * KV_PAGE + (pos % KV_PAGE)) * (a.v_row ? a.v_row : a.dv);
             float inv = 1.f;
             if (a.v_unit) {
                 float ss = 0.f;
@@ -275,6 +281,16 @@ __global__ void attn_prep_kernel(RaggedBatch rb, AttnPrepArgs a) {
             }
             for (int c = lane; c < a.dv; c += 32) kv_store<KT>(dst + c, (src[c] + (bsrc ? bsrc[c] : 0.f)) * inv, a.kv_lo_off);
         }
+    }
+    if (!a.talk) return;
+    __syncthreads();
+    const int rep = a.H / a.G;
+    for (int i = threadIdx.x; i < a.H * a.k_row; i += blockDim.x) {
+        const int h = i / a.k_row, cc = i - h * a.k_row, g = cc / a.d, c = cc - g * a.d;
+        float v = 0.f;
+        if (g < a.G)
+            for (int j = g * rep; j < (g + 1) * rep; ++j) v = fmaf(a.talk[h * a.H + j], sq[j * a.d + c], v);
+        store_act(a.q_out, r, i, v);
     }
 }
 
@@ -341,7 +357,7 @@ __global__ void __launch_bounds__(AC_WARPS * 32) attn_conv_prep_kernel(RaggedBat
 }
 
 constexpr int ATT_WARPS = 4;
-constexpr int ATT_MAXC = 8;      // value columns per lane: dv <= 256
+constexpr int ATT_MAXC = 16;     // most value columns per lane: dv <= 512 (kernels are compiled for 8 and 16)
 
 // Block = (row, group of up to REP query heads that share one key/value head, split).  Its warps walk 32-key tiles of the split's
 // key range: one key per lane for the scores -- the key is fetched and widened once and multiplied into every query head of the
@@ -367,7 +383,7 @@ __device__ __forceinline__ float attn_out_factor(const SinkAttnArgs& a, int r, i
     if (!a.gate) return a.out_mult;
     return a.out_mult / (1.f + __expf(-a.gate[(size_t)r * a.ldg + (a.gate_heads ? h : h * a.dv + col)]));
 }
-template <typename KT, int REP, bool STAGE>
+template <typename KT, int REP, bool STAGE, int MAXC>
 __global__ void __launch_bounds__(ATT_WARPS * 32) sink_attention_kernel(RaggedBatch rb, SinkAttnArgs a) {
     constexpr bool stage = STAGE;
     extern __shared__ __align__(16) float smem[];
@@ -389,21 +405,22 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) sink_attention_kernel(RaggedBa
     const int nkt = min((keep + 31) / 32, t0);           // their tiles come first, those that the window does not reach
     const int ntiles = (nkeys + 31) / 32, per = (nkt + ntiles - t0 + a.nsplit - 1) / a.nsplit;
     const int t_lo = sp * per, t_hi = min(nkt + ntiles - t0, t_lo + per);
-    float m[REP], l[REP], acc[REP][ATT_MAXC];
+    float m[REP], l[REP], acc[REP][MAXC];
 #pragma unroll
     for (int q = 0; q < REP; ++q) {
         m[q] = -INFINITY; l[q] = 0.f;
 #pragma unroll
-        for (int c = 0; c < ATT_MAXC; ++c) acc[q][c] = 0.f;
+        for (int c = 0; c < MAXC; ++c) acc[q][c] = 0.f;
     }
-    const bool kvec = (d & 7) == 0, vvec = (dv & 7) == 0;
+    const int v_row = a.v_row ? a.v_row : dv, Gk = a.Gk ? a.Gk : a.G, gk = h0 / (a.H / Gk);
+    const bool kvec = (d & 7) == 0, vvec = (dv & 7) == 0 && (v_row & 7) == 0;
     // STAGE (widths that allow 16-byte copies, room in shared memory, a small launch): a warp first brings its whole tile -- 32 key rows and
     // 32 value rows, every plane -- into its own shared-memory patch with one burst of cp.async, so the tile costs one trip to memory
     // instead of a dozen dependent load rounds; rows are padded by 16 bytes, which spreads a lane-per-row access over all banks.
     // The arithmetic and its order are the same either way.
-    // kv_shared (one pool serves as keys and as values, d == dv): the staged key rows are the value rows too -- one copy, half the patch.
+    // kv_shared (one pool serves as keys and as values): the staged key rows are the value rows too -- one copy, half the patch.
     const bool one_copy = stage && a.kv_shared;
-    const int ks_e = stage ? d + 16 / (int)sizeof(KT) : d, vs_e = stage ? dv + 16 / (int)sizeof(KT) : dv;      // row strides (elements)
+    const int ks_e = stage ? d + 16 / (int)sizeof(KT) : d, vs_e = !stage ? v_row : one_copy ? ks_e : dv + 16 / (int)sizeof(KT);      // row strides (elements)
     const int planes = (sizeof(KT) == 2 && a.kv_lo_off) ? 2 : 1;
     KT* kst = nullptr; KT* vst = nullptr;
     if (stage) {
@@ -416,14 +433,14 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) sink_attention_kernel(RaggedBa
         const int t = ti < nkt ? ti : t0 + ti - nkt;
         const int j = t * 32 + lane;
         const int pg = bt[(t * 32) / KV_PAGE];           // a 32-key tile never straddles a 64-token page
-        const size_t base = ((size_t)pg * a.G + g) * KV_PAGE + ((t * 32) % KV_PAGE);
+        const size_t base = ((size_t)pg * Gk + gk) * KV_PAGE + ((t * 32) % KV_PAGE), vbase = ((size_t)pg * a.G + g) * KV_PAGE + ((t * 32) % KV_PAGE);
         const int cnt = min(32, nkeys - t * 32);
         if (stage) {
             __syncwarp();                                 // the patch's last readers are done
             const int kc = d * (int)sizeof(KT) / 16, vc = dv * (int)sizeof(KT) / 16;      // 16-byte pieces per row
             for (int pl = 0; pl < planes; ++pl) {
                 const KT* ksrc = (const KT*)a.k_pool + base * d + (pl ? a.kv_lo_off : 0);
-                const KT* vsrc = (const KT*)a.v_pool + base * dv + (pl ? a.kv_lo_off : 0);
+                const KT* vsrc = (const KT*)a.v_pool + vbase * v_row + (pl ? a.kv_lo_off : 0);
                 for (int i = lane; i < cnt * kc; i += 32) {
                     const int row = i / kc, ch = i % kc;
                     cp_async16s(reinterpret_cast<unsigned char*>(kst + (size_t)pl * 32 * ks_e + (size_t)row * ks_e) + ch * 16,
@@ -432,7 +449,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) sink_attention_kernel(RaggedBa
                 for (int i = lane; i < (one_copy ? 0 : cnt * vc); i += 32) {
                     const int row = i / vc, ch = i % vc;
                     cp_async16s(reinterpret_cast<unsigned char*>(vst + (size_t)pl * 32 * vs_e + (size_t)row * vs_e) + ch * 16,
-                                reinterpret_cast<const unsigned char*>(vsrc + (size_t)row * dv) + ch * 16);
+                                reinterpret_cast<const unsigned char*>(vsrc + (size_t)row * v_row) + ch * 16);
                 }
             }
             asm volatile("cp.async.commit_group;\n cp.async.wait_group 0;" ::: "memory");
@@ -497,17 +514,19 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) sink_attention_kernel(RaggedBa
             p[q] = seen ? __expf(sv - mn) : 0.f;
             l[q] = l[q] * corr + warp_sum(p[q]);
 #pragma unroll
-            for (int c = 0; c < ATT_MAXC; ++c) acc[q][c] *= corr;
+            for (int c = 0; c < MAXC; ++c) acc[q][c] *= corr;
             m[q] = mn;
         }
-        const KT* vb = stage ? vst : (const KT*)a.v_pool + base * dv;
+        const KT* vb = stage ? vst : (const KT*)a.v_pool + vbase * v_row;
         if (vvec) {
-            const bool mine = 8 * lane < dv;
+#pragma unroll
+            for (int hf = 0; hf < MAXC / 8; ++hf) {           // (columns 8 lane .. and, from 257 on, 256 + 8 lane ..)
+            const bool mine = 8 * lane + 256 * hf < dv;
             constexpr int VN = REP <= 2 ? 4 : 2;              // value rows in flight
             for (int j0 = 0; j0 < cnt; j0 += VN) {
                 float v[VN][8];
 #pragma unroll
-                for (int u = 0; u < VN; ++u) if (mine && j0 + u < cnt) kv_load8<KT>(vb + (size_t)(j0 + u) * vs_e + 8 * lane, vlo, v[u]);
+                for (int u = 0; u < VN; ++u) if (mine && j0 + u < cnt) kv_load8<KT>(vb + (size_t)(j0 + u) * vs_e + 8 * lane + 256 * hf, vlo, v[u]);
 #pragma unroll
                 for (int u = 0; u < VN; ++u) {
                     const int jj = j0 + u;                    // (uniform over the warp)
@@ -517,21 +536,22 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) sink_attention_kernel(RaggedBa
                         const float pj = __shfl_sync(0xffffffffu, p[q], jj);
                         if (mine && q < nh) {
 #pragma unroll
-                            for (int c = 0; c < 8; ++c) acc[q][c] = fmaf(pj, v[u][c], acc[q][c]);
+                            for (int c = 0; c < 8; ++c) acc[q][8 * hf + c] = fmaf(pj, v[u][c], acc[q][8 * hf + c]);
                         }
                     }
                 }
             }
+            }
         } else {
             for (int jj = 0; jj < cnt; ++jj) {
-                float v[ATT_MAXC];
+                float v[MAXC];
 #pragma unroll
-                for (int c = 0; c < ATT_MAXC; ++c) { const int col = lane + 32 * c; v[c] = col < dv ? kv_load<KT>(vb + (size_t)jj * dv + col, a.kv_lo_off) : 0.f; }
+                for (int c = 0; c < MAXC; ++c) { const int col = lane + 32 * c; v[c] = col < dv ? kv_load<KT>(vb + (size_t)jj * v_row + col, a.kv_lo_off) : 0.f; }
 #pragma unroll
                 for (int q = 0; q < REP; ++q) {
                     const float pj = __shfl_sync(0xffffffffu, p[q], jj);
 #pragma unroll
-                    for (int c = 0; c < ATT_MAXC; ++c) acc[q][c] = fmaf(pj, v[c], acc[q][c]);
+                    for (int c = 0; c < MAXC; ++c) acc[q][c] = fmaf(pj, v[c], acc[q][c]);
                 }
             }
         }
@@ -542,7 +562,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) sink_attention_kernel(RaggedBa
         if (q < nh) {
             if (lane == 0) { wm[warp * REP + q] = m[q]; wl[warp * REP + q] = l[q]; }
 #pragma unroll
-            for (int c = 0; c < ATT_MAXC; ++c) { const int col = vvec ? 8 * lane + c : lane + 32 * c; if (col < dv) wa[((size_t)warp * REP + q) * dv + col] = acc[q][c]; }
+            for (int c = 0; c < MAXC; ++c) { const int col = vvec ? 8 * lane + (c & 7) + 256 * (c >> 3) : lane + 32 * c; if (col < dv) wa[((size_t)warp * REP + q) * dv + col] = acc[q][c]; }
         }
     }
     __syncthreads();
@@ -1192,7 +1212,8 @@ int linear_f32_launch(cudaStream_t st, const float* A, int lda, const bf16* W, i
                       const float* col_scale, const float* gate, int ldg, const float* gate_bias, const float* bias) {
     if (M <= 0 || N <= 0 || K <= 0) return -1000;
     const dim3 grid((N + 63) / 64, (M + 63) / 64);
-    if (mode == LIN_RESID) linear_f32_kernel<LIN_RESID><<<grid, 256, 0, st>>>(A, lda, W, ldw, M, N, K, C, ldc, col_scale, gate, ldg, gate_bias, bias);
+    if (mode == LIN_RELU2) linear_f32_kernel<LIN_RELU2><<<grid, 256, 0, st>>>(A, lda, W, ldw, M, N, K, C, ldc, nullptr, nullptr, 0, nullptr, nullptr);
+    else if (mode == LIN_RESID) linear_f32_kernel<LIN_RESID><<<grid, 256, 0, st>>>(A, lda, W, ldw, M, N, K, C, ldc, col_scale, gate, ldg, gate_bias, bias);
     else linear_f32_kernel<LIN_STORE><<<grid, 256, 0, st>>>(A, lda, W, ldw, M, N, K, C, ldc, nullptr, nullptr, 0, nullptr, nullptr);
     return last_err();
 }
@@ -1227,14 +1248,20 @@ static int attn_conv_prep_launch(cudaStream_t st, const RaggedBatch& rb, const A
 int attn_prep_launch(cudaStream_t st, const RaggedBatch& rb, const AttnPrepArgs& a) {
     if (a.rot_dims < 0 || (a.rot_dims & 1) || a.rot_dims > a.d || a.rot_dims > 4096) return -1000;
     if (a.v_from_k && a.d != a.dv) return -1000;
-    if (a.rot_halves != (a.conv_w ? 1 : 0) || (a.rot_mag != 1.f && !a.conv_w)) return -1000;
+    if ((a.conv_w && (!a.rot_halves || a.talk)) || (a.rot_mag != 1.f && !a.conv_w)) return -1000;
+    if (a.talk && (a.k_row < a.G * a.d || a.v_from_k || !a.has_kv)) return -1000;
     if (a.conv_w) return a.kv_f32 ? attn_conv_prep_launch<float>(st, rb, a) : attn_conv_prep_launch<bf16>(st, rb, a);
-    const size_t sm = (size_t)a.rot_dims * sizeof(float);
+    const size_t sm = ((size_t)a.rot_dims + (a.talk ? (size_t)a.H * a.d : 0)) * sizeof(float);
+    if (sm > 200 * 1024) return -1000;
+    if (sm > 40 * 1024) {
+        static SmemOptIn seen_f, seen_b;
+        if (const int e = a.kv_f32 ? ensure_dyn_smem(attn_prep_kernel<float>, sm, seen_f) : ensure_dyn_smem(attn_prep_kernel<bf16>, sm, seen_b)) return e;
+    }
     if (a.kv_f32) attn_prep_kernel<float><<<rb.T, 256, sm, st>>>(rb, a);
     else attn_prep_kernel<bf16><<<rb.T, 256, sm, st>>>(rb, a);
     return last_err();
 }
-template <typename KT, int REP>
+template <typename KT, int REP, int MAXC>
 static int sink_attention_launch_t(cudaStream_t st, const RaggedBatch& rb, const SinkAttnArgs& a) {
     const int rep = a.H / a.G, nb = (rep + REP - 1) / REP;
     size_t smem = (size_t)(REP * a.d + 2 * ATT_WARPS * REP + ATT_WARPS * REP * a.dv) * sizeof(float);
@@ -1244,30 +1271,37 @@ static int sink_attention_launch_t(cudaStream_t st, const RaggedBatch& rb, const
     const size_t patch = (size_t)ATT_WARPS * 32 * planes * ((size_t)a.d * sizeof(KT) + 16 + (a.kv_shared ? 0 : (size_t)a.dv * sizeof(KT) + 16)) + 16;
     // ... and the launch is small (a decode step: about two blocks per SM at most).  A launch of thousands of blocks hides its load
     // latency by residency instead, which the patches' shared memory would take away.
-    const int stage = ((a.d & 7) == 0 && (a.dv & 7) == 0 && smem + patch <= 200 * 1024 && (long long)rb.T * a.G * nb * a.nsplit <= 300) ? 1 : 0;
+    const int stage = ((a.d & 7) == 0 && (a.dv & 7) == 0 && (a.v_row & 7) == 0 && smem + patch <= 200 * 1024 && (long long)rb.T * a.G * nb * a.nsplit <= 300) ? 1 : 0;
     if (stage) smem += patch;
     static SmemOptIn seen, seen_staged;
     if (stage) {
-        if (const int e = ensure_dyn_smem(sink_attention_kernel<KT, REP, true>, smem, seen_staged)) return e;
-        sink_attention_kernel<KT, REP, true><<<dim3(rb.T, a.G * nb, a.nsplit), ATT_WARPS * 32, smem, st>>>(rb, a);
+        if (const int e = ensure_dyn_smem(sink_attention_kernel<KT, REP, true, MAXC>, smem, seen_staged)) return e;
+        sink_attention_kernel<KT, REP, true, MAXC><<<dim3(rb.T, a.G * nb, a.nsplit), ATT_WARPS * 32, smem, st>>>(rb, a);
         return last_err();
     }
-    if (const int e = ensure_dyn_smem(sink_attention_kernel<KT, REP, false>, smem, seen)) return e;
-    sink_attention_kernel<KT, REP, false><<<dim3(rb.T, a.G * nb, a.nsplit), ATT_WARPS * 32, smem, st>>>(rb, a);
+    if (const int e = ensure_dyn_smem(sink_attention_kernel<KT, REP, false, MAXC>, smem, seen)) return e;
+    sink_attention_kernel<KT, REP, false, MAXC><<<dim3(rb.T, a.G * nb, a.nsplit), ATT_WARPS * 32, smem, st>>>(rb, a);
     return last_err();
 }
 template <typename KT>
 static int sink_attention_launch_k(cudaStream_t st, const RaggedBatch& rb, const SinkAttnArgs& a) {
     const int rep = a.H / a.G;
     // few blocks (a decode step): one query head per block keeps more SMs busy than sharing the keys would save
-    if (rep == 1 || (long long)rb.T * a.H * a.nsplit <= 1024) return sink_attention_launch_t<KT, 1>(st, rb, a);
-    if (rep == 2) return sink_attention_launch_t<KT, 2>(st, rb, a);
-    if (rep <= 4) return sink_attention_launch_t<KT, 4>(st, rb, a);
-    return sink_attention_launch_t<KT, 8>(st, rb, a);
+    const bool one = rep == 1 || (long long)rb.T * a.H * a.nsplit <= 1024;
+    if (a.dv > 256) {
+        if (one) return sink_attention_launch_t<KT, 1, 16>(st, rb, a);
+        return rep == 2 ? sink_attention_launch_t<KT, 2, 16>(st, rb, a) : sink_attention_launch_t<KT, 4, 16>(st, rb, a);
+    }
+    if (one) return sink_attention_launch_t<KT, 1, 8>(st, rb, a);
+    if (rep == 2) return sink_attention_launch_t<KT, 2, 8>(st, rb, a);
+    if (rep <= 4) return sink_attention_launch_t<KT, 4, 8>(st, rb, a);
+    return sink_attention_launch_t<KT, 8, 8>(st, rb, a);
 }
 int sink_attention_launch(cudaStream_t st, const RaggedBatch& rb, const SinkAttnArgs& a) {
     if (a.dv > 32 * ATT_MAXC || a.H % a.G || a.keep_first < 0) return -1000;
-    if (a.kv_shared && (a.k_pool != a.v_pool || a.d != a.dv)) return -1000;
+    const int v_row = a.v_row ? a.v_row : a.dv;
+    if (a.kv_shared && (a.k_pool != a.v_pool || a.d != v_row)) return -1000;
+    if (v_row < a.dv || (a.Gk && (a.Gk < 1 || a.G % a.Gk))) return -1000;
     int e = a.kv_f32 ? sink_attention_launch_k<float>(st, rb, a) : sink_attention_launch_k<bf16>(st, rb, a);
     if (e || a.nsplit == 1) return e;
     if (a.nsplit > 64) return -1000;

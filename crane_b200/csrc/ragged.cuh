@@ -15,7 +15,8 @@
 //   post-norm residual add (one or two normalised inputs), attention scores with a tanh cap, a logarithmic distance penalty or a
 //   distance table, projection biases, a whole-projection norm, unit-RMS values or values taken from the raw keys (ragged.cu), and,
 //   in ragged_scan.cu, the Mamba-1 selective scan and the mLSTM matrix memory.  In ragged_delta.cu: the gated delta rule with a decay per
-//   head or per key channel, and an embedding of the token that joins behind every layer.
+//   head or per key channel, and an embedding of the token that joins behind every layer.  In ragged_streams.cu: a residual of several
+//   parallel streams; in ragged_lru.cu: the gated linear recurrence with a real decay per channel behind a short convolution.
 #pragma once
 
 #include "common.cuh"
@@ -38,7 +39,7 @@ struct ActOut {
     bf16* hi = nullptr; long long lo_off = 0; int ldb = 0;
 };
 
-enum LinearMode : int { LIN_STORE = 0, LIN_RESID = 1 };
+enum LinearMode : int { LIN_STORE = 0, LIN_RESID = 1, LIN_RELU2 = 2 };      // LIN_RELU2: stores max(v, 0)^2
 
 int embed_scale_rows_launch(cudaStream_t st, const int* ids, int T, const bf16* embed, int W, float scale, float* x, int ldx);
 // x[r, c] = embed[ids[r], c] + (c even ? sin : cos)(row_pos[r] * freq[c / 2]): the embedding row plus a sinusoidal position vector.
@@ -92,7 +93,7 @@ struct AttnPrepArgs {
     int v_from_k = 0;                 // 1: the row has no value columns; the cached value of a head is its key as projected (+ bias), before the norm (dv == d)
     const float* q_head_scale = nullptr;   // nullable [H]: head h's normalised query is multiplied by q_head_scale[h]
     // The form with a short convolution (conv_w != nullptr; no norm, no temperature, no bias; d and dv <= 256):
-    int rot_halves = 0;               // 1, with conv_w only: dimension i turns together with dimension i + rot_dims / 2 (instead of pairs (2i, 2i + 1))
+    int rot_halves = 0;               // 1: dimension i turns together with dimension i + rot_dims / 2 (instead of pairs (2i, 2i + 1))
     float rot_mag = 1.f;              // factor on the rotation's cosines and sines
     // a causal convolution over time on every projected channel (q | k | v columns), ahead of everything else:
     // u_t = sum_j conv_w[c, j] * p_(t - taps + 1 + j), p the projections; inputs ahead of the entry come from the carried window
@@ -100,6 +101,12 @@ struct AttnPrepArgs {
     int conv_taps = 0;
     float* conv_state = nullptr;      // [slots, taps - 1, channels]; moved on here when every entry brings one row, else by causal_conv_window_launch
     int single_rows = 0;
+    // Scores mixed over the heads ahead of the softmax, score_h <- sum_g talk[h, g] score_g (not with conv_w): a mixed score is ONE product
+    // of width G * d, of the row (sum over g in group 0 of talk[h, g] q_g | group 1 | ...) with all key heads of the token side by side.
+    // The queries leave in that form, H rows of k_row >= G * d columns (zeros behind), and the keys of a token are one row of k_row.
+    const float* talk = nullptr;      // [H, H]
+    int k_row = 0;
+    int v_row = 0;                    // row width of a value head's pages (0: dv; columns behind dv stay as they are)
 };
 int attn_prep_launch(cudaStream_t st, const RaggedBatch& rb, const AttnPrepArgs& a);
 
@@ -114,7 +121,7 @@ struct SinkAttnArgs {
     const float* gate; int ldg;       // nullable [T, ldg]: out[r, h * dv + c] *= sigmoid(gate[r, h * dv + c])
     ActOut out;                       // [T, H * dv]
     float* part; int nsplit;          // scratch [T, H, nsplit, dv + 2] when nsplit > 1
-    int kv_shared = 0;                // 1: k_pool == v_pool and d == dv -- a cached row is its own value (staged once)
+    int kv_shared = 0;                // 1: k_pool == v_pool -- a cached row, or the first dv columns of it, is its own value (staged once)
     // score modifiers, applied in this order after the scale: s <- softcap * tanh(s / softcap) (softcap > 0);
     // s <- s - dist_r1[h] * ln(1 + dist_r2[h] * (i - j)) (dist_r1 != nullptr);  s <- s + dist_table[h * dist_rows + min(i - j, dist_rows - 1)]
     float softcap = 0.f;
@@ -123,6 +130,8 @@ struct SinkAttnArgs {
     int keep_first = 0;                      // window > 0: the first keep_first tokens of the sequence stay visible behind the window
     int gate_heads = 0;                      // 1: gate is [T, ldg] with one number per head: out[r, h * dv + c] *= sigmoid(gate[r, h])
     float out_mult = 1.f;                    // factor on every output
+    int Gk = 0;                              // key heads in k_pool (0: G): head h reads key head h / (H / Gk) and value head h / (H / G); G % Gk == 0
+    int v_row = 0;                           // row width of v_pool (0: dv).  kv_shared: v_row == d, a cached row's first dv columns are its value
 };
 int sink_attention_launch(cudaStream_t st, const RaggedBatch& rb, const SinkAttnArgs& a);
 
@@ -233,9 +242,42 @@ struct LatentPrepArgs {
 };
 int latent_prep_launch(cudaStream_t st, const RaggedBatch& rb, const LatentPrepArgs& a);
 
+// Latent attention whose queries and keys carry a rotated part beside the latent one.  proj [T, ld]: H x (dim | rot_dim) queries, kv_rank
+// latent columns, rot_dim columns of one key part shared by the heads.  The latent is RMS-normed with its weight; the rotated parts turn in
+// pairs (2i, 2i + 1) of their first rot_dims dimensions by pos * rot_freq[i].  latent | rotated key goes to the sequence's page as one row of
+// row_w >= kv_rank + rot_dim columns.  Of the queries, head h's row of q_out (q_w columns) receives the rotated part at column rot_col
+// (zeros behind it) and, with whole_q, the unrotated part at its start (rot_col == dim).
+struct LatentRotArgs {
+    const float* proj; int ld;
+    int H, dim, rot_dim, kv_rank;
+    const float* kv_w; float eps;
+    int rot_dims; const double* rot_freq;
+    void* pool; int kv_f32; long long kv_lo_off; int row_w;
+    const int* block_table; int max_pages;
+    ActOut q_out; int q_w, rot_col, whole_q;
+};
+int latent_rot_prep_launch(cudaStream_t st, const RaggedBatch& rb, const LatentRotArgs& a);
+
+// Keys and values of every head built from cached latent rows.  The rows that the step's queries can see (per entry the `reach` tokens
+// before it -- fewer where the sequence is shorter -- and its own) are numbered entry by entry; `gather` copies latents i0 .. i0 + n - 1 into a
+// linear's operand, `scatter` takes the linear's rows (H x dim keys | H x dv values) to scratch pages: keys [n_pages, H, KV_PAGE, k_w] with the
+// shared rotated part behind each head's own, values [n_pages, H, KV_PAGE, v_w].  bf16 pages only.
+struct LatentBuildArgs {
+    const bf16* pool; long long kv_lo_off; int row_w, kv_rank, rot_dim;
+    const int* block_table; int max_pages;
+    int reach;
+    int H, dim, dv;
+    ActOut ckv;                       // planes [n, .. kv_rank]
+    const float* kv; int ld;          // [n, ld]
+    bf16* k_out; bf16* v_out; long long out_lo; int k_w, v_w;
+};
+int latent_gather_launch(cudaStream_t st, const RaggedBatch& rb, const LatentBuildArgs& a, int i0, int n);
+int latent_scatter_launch(cudaStream_t st, const RaggedBatch& rb, const LatentBuildArgs& a, int i0, int n);
+
 // Block-diagonal linear: out[r, h * n_out + i] = sum_j in[r, h * n_in + j] * w[(h * n_in + j) * n_out + i], every product and sum in
 // f32 in the order j = 0, 1, ...  (w is stored input-major per head: [H, n_in, n_out] bf16).
-int headwise_linear_launch(cudaStream_t st, const ActOut& in, const bf16* w, int T, int H, int n_in, int n_out, const ActOut& out);
+// in_w / out_w: columns from one head's slice to the next in `in` / `out` (0: n_in / n_out).
+int headwise_linear_launch(cudaStream_t st, const ActOut& in, const bf16* w, int T, int H, int n_in, int n_out, const ActOut& out, int in_w = 0, int out_w = 0);
 
 // Gated linear attention.  proj [T, ld] holds q | k | v | g | a (H*d, H*d, H*dv, H*dv, rank columns).  Per head and key channel the
 // decay is sigmoid(z)^(1 / tau), z = a2 a + b (all f32); S_t = diag(decay_t) S_(t-1) + k_t v_t^T; o_t = S_t^T (q_t * q_scale); then
@@ -359,6 +401,46 @@ int token_gate_launch(cudaStream_t st, const float* z, int ldz, int T, int n, co
 // ... with z = x w^T taken in the same launch, for a few rows: x [T, ldx] f32, w [n, ldw] bf16, K (multiple of 8) columns
 int token_gate_step_launch(cudaStream_t st, const float* x, int ldx, const bf16* w, int ldw, int K, int T, int n, const int* ids, const bf16* table, int ldt,
                            int col0, const ActOut& out);
+
+// ---- a residual of parallel streams (ragged_streams.cu) ------------------------------------------------------------------------------------
+// xs [T, S, ldx]: S copies of the stream per row.  One pass per row: the pending sublayer output joins (y != nullptr: x_t <- sum_s mix[s, t] x_s +
+// out[t] y, all copies from the old ones), the copies are summed with the weights `in` (nullptr: ones), and the sum's RMS norm times norm_w
+// leaves as h.  ids: the copies start as the token's embedding row (instead of being read).  store: the new copies are written back.
+// rows: gather list of h's rows (nullptr: identity).
+struct StreamArgs {
+    float* xs; int ldx; int S, W;
+    const int* rows;
+    const int* ids; const bf16* embed;
+    const float* y; int ldy; const float* mix; const float* out;
+    int store;
+    const float* in; const float* norm_w; float eps;
+    ActOut h;
+};
+constexpr int STREAM_MAX = 8, STREAM_MAX_W = 8192;
+int stream_rows_launch(cudaStream_t st, const StreamArgs& a, int R);
+
+// ---- gated linear recurrence with a real decay per channel (ragged_lru.cu) -----------------------------------------------------------------
+// proj [T, ld] holds two branches of `width` columns, from y_col and x_col on.  Per channel and token, all in f32:
+//   u = conv(x + x_b) + conv_b  (causal, `taps` taps, carried);  r, i = sigmoid(block-diagonal linear of u + r_b / i_b), `blocks` equal parts
+//   a = exp(-rate r);  S <- a S + sqrt(1 - a^2) i u;  out = out_mult * S gelu_tanh(y + y_b)
+// State: S [slots, width] and the last `taps` inputs, a ring [slots, taps, width] indexed by the position.
+struct LruArgs {
+    const float* proj; int ld, y_col, x_col;
+    int width, blocks, taps;
+    const float *y_b, *x_b, *conv_w, *conv_b;
+    const bf16* w_gates;              // [blocks][column tiles][pad32(n)][LRU_TILE_COLS r | LRU_TILE_COLS i], n = width / blocks: input-major, zero-padded
+    const float *r_b, *i_b, *rate;    // [width]
+    float *ring, *state;
+    float *dec, *gin, *agg, *next;    // scratch: [T, width] x 2, lru_agg_floats(T, E, width), [E, width]
+    ActOut out; int out_col; float out_mult;
+    int single_rows;                  // every entry brings one row
+    int exact;                        // the gates' products in f32 on CUDA cores
+};
+constexpr int LRU_TILE_COLS = 64;
+size_t lru_gate_weights(int width, int blocks);
+size_t lru_agg_floats(int rows, int entries, int width);
+int lru_mixer_launch(cudaStream_t st, const RaggedBatch& rb, const LruArgs& a);
+int lru_launch_count(const LruArgs& a);
 
 // dst[r, c] = cap * tanh(src[r, c] / cap) for c < V (cap <= 0: a plain copy)
 int softcap_rows_launch(cudaStream_t st, const float* src, int lds, int R, int V, float cap, float* dst, int ldd);

@@ -102,6 +102,96 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(RaggedBatch rb, Latent
     }
 }
 
+// Latent attention with a rotated part, block per row: the latent's norm (thread-strided sum of squares, warp tree, warps in order), the
+// shared key part's rotation, both into the row's page; the queries' parts to where the products read them.  The row's cosines and sines
+// are taken once, in 64-bit.
+template <typename KT>
+__global__ void __launch_bounds__(256) latent_rot_prep_kernel(RaggedBatch rb, LatentRotArgs a) {
+    extern __shared__ float lcs[];                        // [rot_dims / 2] cos, then sin
+    __shared__ float red[8];
+    const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nrot = a.rot_dims / 2;
+    const int e = rb.row_entry[r], pos = rb.row_pos[r], slot = rb.ent_slot[e];
+    const int page = a.block_table[(size_t)slot * a.max_pages + pos / KV_PAGE];
+    KT* dst = (KT*)a.pool + ((size_t)page * KV_PAGE + (pos % KV_PAGE)) * a.row_w;
+    const float* q = a.proj + (size_t)r * a.ld;
+    const float* low = q + (size_t)a.H * (a.dim + a.rot_dim);
+    for (int i = threadIdx.x; i < nrot; i += 256) {
+        double sn, cs;
+        sincos((double)pos * a.rot_freq[i], &sn, &cs);
+        lcs[i] = (float)cs; lcs[nrot + i] = (float)sn;
+    }
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < a.kv_rank; c += 256) ss = fmaf(low[c], low[c], ss);
+    ss = warp_sum(ss);
+    if (lane == 0) red[warp] = ss;
+    __syncthreads();
+    float tot = 0.f;
+#pragma unroll
+    for (int k = 0; k < 8; ++k) tot += red[k];
+    const float inv = 1.f / sqrtf(tot / (float)a.kv_rank + a.eps);
+    for (int c = threadIdx.x; c < a.kv_rank; c += 256) kv_store<KT>(dst + c, low[c] * inv * a.kv_w[c], a.kv_lo_off);
+    auto turned = [&](const float* v, int i) {            // dimension i of a rotated part
+        if (i >= 2 * nrot) return v[i];
+        const float cs = lcs[i >> 1], sn = lcs[nrot + (i >> 1)];
+        return (i & 1) ? v[i] * cs + v[i - 1] * sn : v[i] * cs - v[i + 1] * sn;
+    };
+    for (int i = threadIdx.x; i < a.rot_dim; i += 256) kv_store<KT>(dst + a.kv_rank + i, turned(low + a.kv_rank, i), a.kv_lo_off);
+    const int c0 = a.whole_q ? 0 : a.rot_col, n = a.q_w - c0;
+    for (int i = threadIdx.x; i < a.H * n; i += 256) {
+        const int h = i / n, c = c0 + i - h * n;
+        const float* qh = q + (size_t)h * (a.dim + a.rot_dim);
+        const float v = c < a.rot_col ? qh[c] : c < a.rot_col + a.rot_dim ? turned(qh + a.dim, c - a.rot_col) : 0.f;
+        store_act(a.q_out, r, h * a.q_w + c, v);
+    }
+}
+
+// Number i of the rows a step's queries can see -> the sequence slot and the position.
+__device__ __forceinline__ bool seen_row(const RaggedBatch& rb, int reach, int i, int& slot, int& pos) {
+    for (int e = 0; e < rb.E; ++e) {
+        const int p0 = rb.ent_pos0[e], back = min(p0, reach), n = back + rb.ent_len[e];
+        if (i < n) { slot = rb.ent_slot[e]; pos = p0 - back + i; return true; }
+        i -= n;
+    }
+    return false;
+}
+__global__ void __launch_bounds__(128) latent_gather_kernel(RaggedBatch rb, LatentBuildArgs a, int i0) {
+    int slot, pos;
+    if (!seen_row(rb, a.reach, i0 + blockIdx.x, slot, pos)) return;
+    const int page = a.block_table[(size_t)slot * a.max_pages + pos / KV_PAGE];
+    const bf16* src = a.pool + ((size_t)page * KV_PAGE + pos % KV_PAGE) * a.row_w;
+    bf16* dst = a.ckv.hi + (size_t)blockIdx.x * a.ckv.ldb;
+    const int pieces = (a.kv_rank & 7) ? 0 : a.kv_rank / 8;      // 16-byte pieces where the rank allows
+    for (int p = 0; p < (a.kv_lo_off ? 2 : 1); ++p) {
+        const bf16* s = src + (p ? a.kv_lo_off : 0);
+        bf16* d = dst + (p ? a.ckv.lo_off : 0);
+        for (int c = threadIdx.x; c < pieces; c += 128) reinterpret_cast<uint4*>(d)[c] = reinterpret_cast<const uint4*>(s)[c];
+        if (!pieces) for (int c = threadIdx.x; c < a.kv_rank; c += 128) d[c] = s[c];
+    }
+}
+__global__ void __launch_bounds__(256) latent_scatter_kernel(RaggedBatch rb, LatentBuildArgs a, int i0) {
+    int slot, pos;
+    if (!seen_row(rb, a.reach, i0 + blockIdx.x, slot, pos)) return;
+    const int page = a.block_table[(size_t)slot * a.max_pages + pos / KV_PAGE], at = pos % KV_PAGE;
+    const float* kv = a.kv + (size_t)blockIdx.x * a.ld;
+    const bf16* rot = a.pool + ((size_t)page * KV_PAGE + at) * a.row_w + a.kv_rank;
+    const int kn = a.dim + a.rot_dim, C = a.H * a.dim;
+    auto put = [&](bf16* d, float v) {
+        const bf16 h = __float2bfloat16_rn(v);
+        *d = h;
+        if (a.out_lo) d[a.out_lo] = __float2bfloat16_rn(v - __bfloat162float(h));
+    };
+    for (int i = threadIdx.x; i < a.H * kn; i += 256) {
+        const int h = i / kn, c = i - h * kn;
+        bf16* d = a.k_out + (((size_t)page * a.H + h) * KV_PAGE + at) * a.k_w + c;
+        if (c < a.dim) put(d, kv[h * a.dim + c]);
+        else { *d = rot[c - a.dim]; if (a.out_lo) d[a.out_lo] = rot[a.kv_lo_off + c - a.dim]; }
+    }
+    for (int i = threadIdx.x; i < a.H * a.dv; i += 256) {
+        const int h = i / a.dv, c = i - h * a.dv;
+        put(a.v_out + (((size_t)page * a.H + h) * KV_PAGE + at) * a.v_w + c, kv[C + i]);
+    }
+}
+
 // Block = (HW_ROWS rows, head): the rows' input slices sit in shared memory, a thread owns output columns i, i + 128, ... and walks the
 // head's [n_in, n_out] matrix down its column (neighbouring threads read neighbouring weights).
 constexpr int HW_ROWS = 8;
@@ -110,12 +200,12 @@ __device__ __forceinline__ float act_load(const ActOut& o, int r, int c) {
     const bf16* p = o.hi + (size_t)r * o.ldb + c;
     return __bfloat162float(*p) + (o.lo_off ? __bfloat162float(p[o.lo_off]) : 0.f);
 }
-__global__ void __launch_bounds__(128) headwise_linear_kernel(ActOut in, const bf16* __restrict__ w, int T, int n_in, int n_out, ActOut out) {
+__global__ void __launch_bounds__(128) headwise_linear_kernel(ActOut in, const bf16* __restrict__ w, int T, int n_in, int n_out, ActOut out, int in_w, int out_w) {
     extern __shared__ float hw_in[];                      // [HW_ROWS][n_in]
     const int r0 = blockIdx.x * HW_ROWS, h = blockIdx.y, nr = min(HW_ROWS, T - r0);
     for (int i = threadIdx.x; i < HW_ROWS * n_in; i += blockDim.x) {
         const int rr = i / n_in, j = i - rr * n_in;
-        hw_in[i] = rr < nr ? act_load(in, r0 + rr, h * n_in + j) : 0.f;
+        hw_in[i] = rr < nr ? act_load(in, r0 + rr, h * in_w + j) : 0.f;
     }
     __syncthreads();
     const bf16* wh = w + (size_t)h * n_in * n_out;
@@ -129,7 +219,7 @@ __global__ void __launch_bounds__(128) headwise_linear_kernel(ActOut in, const b
             for (int rr = 0; rr < HW_ROWS; ++rr) acc[rr] = fmaf(hw_in[rr * n_in + j], wv, acc[rr]);
         }
 #pragma unroll
-        for (int rr = 0; rr < HW_ROWS; ++rr) if (rr < nr) store_act(out, r0 + rr, h * n_out + i, acc[rr]);
+        for (int rr = 0; rr < HW_ROWS; ++rr) if (rr < nr) store_act(out, r0 + rr, h * out_w + i, acc[rr]);
     }
 }
 
@@ -137,12 +227,12 @@ __global__ void __launch_bounds__(128) headwise_linear_kernel(ActOut in, const b
 // them, a lane owns four neighbouring columns (one 8-byte load of the bf16 weights per input row, the warp reads 256 contiguous bytes;
 // a warp's handful of rows are all requested before the first is used), and the warps' partial sums meet in warp order.
 constexpr int HWF_ROWS = 4, HWF_WARPS = 16, HWF_COLS = 128;
-__global__ void __launch_bounds__(HWF_WARPS * 32) headwise_few_kernel(ActOut in, const bf16* __restrict__ w, int T, int n_in, int n_out, ActOut out) {
+__global__ void __launch_bounds__(HWF_WARPS * 32) headwise_few_kernel(ActOut in, const bf16* __restrict__ w, int T, int n_in, int n_out, ActOut out, int in_w, int out_w) {
     extern __shared__ float hwf_s[];                      // [T][n_in] inputs, then [warps][HWF_ROWS][HWF_COLS] partial sums
     float* xin = hwf_s;
     float* part = hwf_s + (((size_t)T * n_in + 3) & ~(size_t)3);
     const int h = blockIdx.y, c0 = blockIdx.x * HWF_COLS, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int i = threadIdx.x; i < T * n_in; i += blockDim.x) { const int rr = i / n_in, j = i - rr * n_in; xin[i] = act_load(in, rr, h * n_in + j); }
+    for (int i = threadIdx.x; i < T * n_in; i += blockDim.x) { const int rr = i / n_in, j = i - rr * n_in; xin[i] = act_load(in, rr, h * in_w + j); }
     __syncthreads();
     const int col = c0 + 4 * lane, per = (n_in + HWF_WARPS - 1) / HWF_WARPS, j0 = warp * per, j1 = min(n_in, j0 + per);
     const bool vec = (n_out & 3) == 0;                     // (then every group of four starts on an 8-byte boundary)
@@ -182,7 +272,7 @@ __global__ void __launch_bounds__(HWF_WARPS * 32) headwise_few_kernel(ActOut in,
         float sum = 0.f;
 #pragma unroll
         for (int wq = 0; wq < HWF_WARPS; ++wq) sum += part[((size_t)wq * HWF_ROWS + rr) * HWF_COLS + c];
-        store_act(out, rr, h * n_out + c0 + c, sum);
+        store_act(out, rr, h * out_w + c0 + c, sum);
     }
 }
 
@@ -478,19 +568,39 @@ int latent_prep_launch(cudaStream_t st, const RaggedBatch& rb, const LatentPrepA
     else latent_prep_kernel<bf16><<<rb.T, 256, 0, st>>>(rb, a);
     return last_err();
 }
-int headwise_linear_launch(cudaStream_t st, const ActOut& in, const bf16* w, int T, int H, int n_in, int n_out, const ActOut& out) {
+int latent_rot_prep_launch(cudaStream_t st, const RaggedBatch& rb, const LatentRotArgs& a) {
+    if (a.kv_rank < 1 || a.rot_dim < 0 || a.rot_dims < 0 || (a.rot_dims & 1) || a.rot_dims > a.rot_dim || a.rot_dims > 4096 || a.row_w < a.kv_rank + a.rot_dim ||
+        a.q_w < a.rot_col + a.rot_dim || (a.whole_q && a.rot_col != a.dim)) return -1000;
+    const size_t sm = (size_t)a.rot_dims * sizeof(float);
+    if (a.kv_f32) latent_rot_prep_kernel<float><<<rb.T, 256, sm, st>>>(rb, a);
+    else latent_rot_prep_kernel<bf16><<<rb.T, 256, sm, st>>>(rb, a);
+    return last_err();
+}
+int latent_gather_launch(cudaStream_t st, const RaggedBatch& rb, const LatentBuildArgs& a, int i0, int n) {
+    if (n < 1 || !a.ckv.hi || (a.kv_lo_off != 0) != (a.ckv.lo_off != 0) || (a.row_w & 7) || (a.ckv.ldb & 7)) return -1000;
+    latent_gather_kernel<<<n, 128, 0, st>>>(rb, a, i0);
+    return last_err();
+}
+int latent_scatter_launch(cudaStream_t st, const RaggedBatch& rb, const LatentBuildArgs& a, int i0, int n) {
+    if (n < 1 || a.k_w < a.dim + a.rot_dim || a.v_w < a.dv || (a.kv_lo_off != 0) != (a.out_lo != 0)) return -1000;
+    latent_scatter_kernel<<<n, 256, 0, st>>>(rb, a, i0);
+    return last_err();
+}
+int headwise_linear_launch(cudaStream_t st, const ActOut& in, const bf16* w, int T, int H, int n_in, int n_out, const ActOut& out, int in_w, int out_w) {
+    if (!in_w) in_w = n_in;
+    if (!out_w) out_w = n_out;
     const size_t smem = (size_t)HW_ROWS * n_in * sizeof(float);
     if ((!in.f && !in.hi) || smem > 200 * 1024) return -1000;
     if (T <= HWF_ROWS) {
         const size_t sf = ((size_t)((T * n_in + 3) & ~3) + (size_t)HWF_WARPS * HWF_ROWS * HWF_COLS) * sizeof(float);
         static SmemOptIn seen_few;
         if (const int e = ensure_dyn_smem(headwise_few_kernel, sf, seen_few)) return e;
-        headwise_few_kernel<<<dim3((n_out + HWF_COLS - 1) / HWF_COLS, H), HWF_WARPS * 32, sf, st>>>(in, w, T, n_in, n_out, out);
+        headwise_few_kernel<<<dim3((n_out + HWF_COLS - 1) / HWF_COLS, H), HWF_WARPS * 32, sf, st>>>(in, w, T, n_in, n_out, out, in_w, out_w);
         return last_err();
     }
     static SmemOptIn seen;
     if (const int e = ensure_dyn_smem(headwise_linear_kernel, smem, seen)) return e;
-    headwise_linear_kernel<<<dim3((T + HW_ROWS - 1) / HW_ROWS, H), 128, smem, st>>>(in, w, T, n_in, n_out, out);
+    headwise_linear_kernel<<<dim3((T + HW_ROWS - 1) / HW_ROWS, H), 128, smem, st>>>(in, w, T, n_in, n_out, out, in_w, out_w);
     return last_err();
 }
 int gla_launch_count(bool has_seg_scratch, int max_len) { return has_seg_scratch && max_len >= GLA_SEG_MIN ? 5 : 3; }
