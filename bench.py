@@ -718,7 +718,7 @@ def layer_list_work(cfg, S, n_dec):
     shapes = {n: sh for n, sh, k in synth.tensor_specs(cfg)}
     per_tok, attn_fl, cache_b = V * W, 0.0, 0.0
     for i, L in enumerate(cfg["layers"]):
-        per_tok += sum(sh[0] * sh[1] for n, sh in shapes.items() if n.startswith(f"l{i}.") and len(sh) == 2 and ".mix.conv" not in n and not n.endswith(".conv"))
+        per_tok += sum(int(np.prod(sh)) for n, sh in shapes.items() if n.startswith(f"l{i}.") and len(sh) >= 2 and ".mix.conv" not in n and not n.endswith((".conv", "ra.b", "ri.b")))
         a = L["mixer"]
 
         def attention(a):
@@ -727,6 +727,12 @@ def layer_list_work(cfg, S, n_dec):
             return 2.0 * S * keys * a["heads"] * (a["dim"] + a["vdim"]), ctx * a["kv_heads"] * (a["dim"] + a["vdim"]) * 4
         if L["type"] == "attention":
             f, b = attention(a)
+        elif L["type"] == "latent_attention":          # scores and sums at the heads' own widths; one latent row (hi + lo planes) per cached token
+            keys, ctx = min(S / 2, a["mask"]["size"]), min(S + n_dec / 2, a["mask"]["size"])
+            f, b = 2.0 * S * keys * a["heads"] * (a["dim"] + a["rot_dim"] + a["vdim"]), ctx * (a["kv_rank"] + a["rot_dim"]) * 4
+        elif L["type"] == "parallel" and "blocks" in a["right"]:       # beside a linear recurrence with a state per channel
+            f, b = attention(a["left"])
+            b += 2 * 4 * a["right"]["width"] * (1 + a["right"]["conv"])
         elif L["type"] == "parallel":
             f, b = attention(a["left"])
             r = a["right"]
@@ -901,6 +907,72 @@ def bench_suvapel(args, rank, world, local_rank):
     print(json.dumps(out))
 
 
+def bench_rupulix(args, rank, world, local_rank):
+    """The Rupulix layer-list decoder (two parallel residual streams; windowed latent attention with a rotated part and a sink; attention with
+    mixed scores and no window beside a gated linear recurrence; squared-ReLU feed-forward) beside the closest existing model, a Puzonex
+    stack with windowed sink attention where Rupulix has latent attention and attention without a window beside a matrix memory where it
+    has its parallel mixer, at equal width, depth, heads, windows and feed-forward weights (a gated unit of two thirds of the width), at two
+    sizes.  One request = 4096-token prefill + 256 greedy tokens through `crane_b200_generate_greedy`; one GPU."""
+    if args.impl == "reference":
+        if rank == 0:
+            print(json.dumps({"impl": "reference", "unavailable": "the reference has no model of this design"}))
+        return
+    if rank != 0:
+        return
+    import crane_b200
+    S, n_dec = 4096, 256
+    peaks = load_peaks()
+    sampler = ClockSampler(0)
+
+    def closest(**kw):
+        c = synth.puzonex_config(**kw)
+        _, par, att = c["layers"][:3]
+        par = json.loads(json.dumps(par))
+        par["mixer"]["left"].pop("mask")
+        c["layers"] = [json.loads(json.dumps(par if i % 3 == 2 else att)) for i in range(len(c["layers"]))]
+        return c
+    sizes = {
+        "w1024_12layers_ff5376": dict(
+            rpx=synth.rupulix_config(width=1024, layers=12, heads=8, kv_rank=256, window=1024, kv_heads=2, dim=128, vdim=128, lru_width=1024, lru_blocks=8, ff=5376),
+            pzx=closest(width=1024, layers=12, heads=8, kv_heads=2, dim=128, window=1024, mem_heads=4, mem_dim=128, mem_vdim=256, ff=3584)),
+        "w2048_9layers_ff8448": dict(
+            rpx=synth.rupulix_config(width=2048, layers=9, heads=16, kv_rank=512, window=2048, kv_heads=2, dim=128, vdim=128, lru_width=2048, lru_blocks=8, ff=8448),
+            pzx=closest(width=2048, layers=9, heads=16, kv_heads=2, dim=128, window=2048, mem_heads=8, mem_dim=128, mem_vdim=256, bias_max=2048, ff=5632)),
+    }
+    only = os.environ.get("CRANE_B200_BENCH_ONLY", "")          # "rupulix" / "closest": one side only (launch lists, profiles)
+    cut = int(os.environ.get("CRANE_B200_BENCH_LAYERS", "0"))   # with it: that many layers only
+    variants = {}
+    sampler.start()
+    for name, pair in sizes.items():
+        variants[name] = {}
+        for key, cls in (("rupulix", crane_b200.RupulixModel), ("closest_model_puzonex", crane_b200.PuzonexModel)):
+            if only and not key.startswith(only):
+                continue
+            cfg = pair["rpx" if key == "rupulix" else "pzx"]
+            if only and cut:
+                cfg["layers"] = cfg["layers"][:cut]
+            m = layer_list_load(cls, cfg, S, n_dec)
+            variants[name][key] = layer_list_measure(m, cfg, name + key, args, peaks, S, n_dec)
+            m.close()
+        if only:
+            break
+    clocks = sampler.summary()
+    first = variants["w1024_12layers_ff5376"]
+    d = first.get("rupulix") or first["closest_model_puzonex"]
+    out = {"metric": "decode_tok_per_s", "unit": "tok/s", "n_gpus": 1, "steps": args.steps, "warmup": max(args.warmup, 3), "higher_is_better": True,
+           "scaling": "weak", "vs_baseline": None, "dtype": "bf16", "data": "synthetic",
+           "config": {"workload": f"Rupulix layer-list decoder (width 1024, 2 streams, 4 x (2 x latent attention, attention beside a linear recurrence), window 1024, feed-forward 5376), {S}-token prefill + {n_dec} greedy decode tokens per request; the closest existing model at equal size beside it",
+                      "weights": "random bf16 blocks (timing only)", "l2": "per-token weight stream > 126 MB L2", "parallelism": "1 GPU",
+                      "precision": os.environ.get("CRANE_B200_PRECISION", "split")},
+           "value": d["decode_tok_s"], "ms_per_step": 1e3 / d["e2e_tok_s"] * n_dec, "prefill_ms": d["prefill_ms"], "prefill_tflops": d["prefill_tflops"],
+           "e2e": {"value": d["e2e_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": int(S * 4), "d2h_bytes_per_step": int((n_dec + 1) * 4),
+                   "api": "crane_b200_generate_greedy (host prompt ids in, host token ids out; prefill inside the timed region)"},
+           "gpu_launches": d["gpu_launches"], "clocks": clocks, "variants": variants,
+           "roofline": {"bound": "hbm", "achieved": d["decode_hbm_gbs"], "peak": peaks["hbm_gbs"], "unit": "GB/s", "frac": d["decode_roofline_frac"],
+                        "peak_source": peaks["source"], "launch": "one decode step (graph replay): the token's weights once + cached rows in reach + recurrent states"}}
+    print(json.dumps(out))
+
+
 def other_config_summary(config, steps=2, timeout_s=120):
     """One more BASELINE config measured by THIS script in a child process (`bench.py --config <config>`), condensed for the headline
     line's `other_configs` field.  A child, so that nothing it does -- a failure, a hang (killed at the timeout) -- can keep the
@@ -929,7 +1001,7 @@ def main():
     ap.add_argument("--steps", type=int, default=5)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="crane_b200", choices=["crane_b200", "reference"])
-    ap.add_argument("--config", default="qwen3_vl_2b", choices=["qwen3_vl_2b", "tiny", "qwen3_8b_q4km", "qwen3_5_0_8b", "fosovik", "gavipel", "nifarax", "puzonex", "suvapel"])
+    ap.add_argument("--config", default="qwen3_vl_2b", choices=["qwen3_vl_2b", "tiny", "qwen3_8b_q4km", "qwen3_5_0_8b", "fosovik", "gavipel", "nifarax", "puzonex", "suvapel", "rupulix"])
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-other-configs", action="store_true", help="skip the config-2 (Qwen3.5-0.8B) child measurement appended to the headline line")
     args = ap.parse_args()
@@ -951,6 +1023,8 @@ def main():
         return bench_puzonex(args, rank, world, local_rank)
     if args.config == "suvapel":
         return bench_suvapel(args, rank, world, local_rank)
+    if args.config == "rupulix":
+        return bench_rupulix(args, rank, world, local_rank)
     cfg = synth.QWEN3_VL_2B if args.config == "qwen3_vl_2b" else synth.TINY_QWEN3_VL
     name = "Qwen3-VL-2B" if args.config == "qwen3_vl_2b" else "tiny-Qwen3-VL"
     workload = f"{name} bf16, 1x(448x448) image + {N_TEXT}-tok prompt, prefill + {N_DECODE} greedy decode tokens per request"

@@ -675,7 +675,63 @@ def suvapel_tensor_specs(cfg: dict):
     yield "head", (V, W), "embed"
 
 
+def rupulix_config(width=1024, vocab=65536, layers=12, heads=8, latent_dim=128, rot_dim=64, latent_vdim=128, kv_rank=256, window=1024, kv_heads=2, dim=128,
+                   vdim=128, lru_width=1024, lru_blocks=8, conv=4, ff=5376, streams=2):
+    """`layers` layers in the order latent attention, latent attention, attention beside a linear recurrence, ..., each with a squared-ReLU
+    feed-forward."""
+    lat = {"heads": heads, "dim": latent_dim, "rot_dim": rot_dim, "vdim": latent_vdim, "kv_rank": kv_rank, "scale": (latent_dim + rot_dim) ** -0.5,
+           "mask": {"size": window}, "rot": {"base": 500000.0, "dims": rot_dim}}
+    par = {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "rot": {"base": 500000.0, "dims": dim}},
+           "right": {"width": lru_width, "blocks": lru_blocks, "conv": conv}, "left_scale": 0.5, "right_scale": 0.5}
+    mlp = {"kind": "dense", "ff": ff} if ff else None
+    ls = [{"type": "parallel" if i % 3 == 2 else "latent_attention", "mixer": dict(par if i % 3 == 2 else lat), "mlp": dict(mlp) if mlp else None} for i in range(layers)]
+    return {"architecture": "Rupulix", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "streams": streams, "logit_scale": 1.0, "layers": ls}
+
+
+def rupulix_tensor_specs(cfg: dict):
+    """(name, shape, kind): 'embed', 'final.norm', 'l<i>.norm1|norm2', 'l<i>.hc1|hc2.in|out|mix', 'l<i>.mlp.up|down', and per mixer
+    'l<i>.mix.q|dkv|dkv.norm|uk|uv|sink|o', or 'l<i>.mix.left.q|k|v|q.norm|k.norm|talk|o' with
+    'l<i>.mix.right.y|y.b|x|x.b|conv|conv.b|ra|ra.b|ri|ri.b|lam|o'."""
+    W, V, n = cfg["width"], cfg["vocab"], cfg["streams"]
+    yield "embed", (V, W), "embed"
+    for i, L in enumerate(cfg["layers"]):
+        p, m = f"l{i}.", L["mixer"]
+        for q in (1, 2) if L.get("mlp") else (1,):
+            yield p + f"norm{q}", (W,), "norm"
+            yield p + f"hc{q}.in", (n,), "stream_in"
+            yield p + f"hc{q}.out", (n,), "norm"
+            yield p + f"hc{q}.mix", (n, n), "near_identity"
+        if L["type"] == "latent_attention":
+            H, d, dr, dv, r = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+            for t, sh in (("q", (H * (d + dr), W)), ("dkv", (r + dr, W)), ("uk", (H * d, r)), ("uv", (H * dv, r)), ("o", (W, H * dv))):
+                yield p + "mix." + t, sh, "linear"
+            yield p + "mix.dkv.norm", (r,), "norm"
+            yield p + "mix.sink", (H,), "bias"
+        else:
+            a, b = m["left"], m["right"]
+            H, G, d, dv, C, k = a["heads"], a["kv_heads"], a["dim"], a["vdim"], b["width"], b["blocks"]
+            for t, sh in (("q", (H * d, W)), ("k", (G * d, W)), ("v", (G * dv, W)), ("o", (W, H * dv))):
+                yield p + "mix.left." + t, sh, "linear"
+            yield p + "mix.left.q.norm", (d,), "norm"
+            yield p + "mix.left.k.norm", (d,), "norm"
+            yield p + "mix.left.talk", (H, H), "near_identity"
+            R = p + "mix.right."
+            for t, sh in (("y", (C, W)), ("x", (C, W)), ("conv", (C, b["conv"])), ("ra", (k, C // k, C // k)), ("ri", (k, C // k, C // k)), ("o", (W, C))):
+                yield R + t, sh, "linear"
+            for t, sh in (("y.b", (C,)), ("x.b", (C,)), ("conv.b", (C,)), ("ra.b", (k, C // k)), ("ri.b", (k, C // k))):
+                yield R + t, sh, "bias"
+            yield R + "lam", (C,), "decay"
+        if L.get("mlp"):
+            F = L["mlp"]["ff"]
+            yield p + "mlp.up", (F, W), "linear"
+            yield p + "mlp.down", (W, F), "linear"
+    yield "final.norm", (W,), "norm"
+
+
 def tensor_specs(cfg: dict):
+    if cfg.get("architecture") == "Rupulix":
+        yield from rupulix_tensor_specs(cfg)
+        return
     if cfg.get("architecture") == "Suvapel":
         yield from suvapel_tensor_specs(cfg)
         return
@@ -726,6 +782,12 @@ def make_tensor(name: str, shape, kind: str) -> np.ndarray:
         x = np.abs(_normal(name, shape, 0.2, 0.5))
     elif kind == "forget_bias":    # forget gates that keep most of a memory
         x = _normal(name, shape, 0.5, 4.0)
+    elif kind == "stream_in":  # weights that sum parallel streams
+        x = _normal(name, shape, 0.05, 1.0 / shape[0])
+    elif kind == "near_identity":
+        x = _normal(name, shape, 0.1) + np.eye(*shape)
+    elif kind == "decay":      # softplus of it times eight is a decay's rate: hundreds of tokens at the small end
+        x = _normal(name, shape, 1.0, -4.5)
     elif kind == "alpha":      # Dynamic-Tanh slope: a scalar near one half
         x = _normal(name, shape, 0.02, 0.5)
     else:
