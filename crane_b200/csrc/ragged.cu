@@ -1304,6 +1304,9 @@ int sink_attention_launch(cudaStream_t st, const RaggedBatch& rb, const SinkAttn
     if (v_row < a.dv || (a.Gk && (a.Gk < 1 || a.G % a.Gk))) return -1000;
     int e = a.kv_f32 ? sink_attention_launch_k<float>(st, rb, a) : sink_attention_launch_k<bf16>(st, rb, a);
     if (e || a.nsplit == 1) return e;
+    return sink_attention_merge_launch(st, rb, a);
+}
+int sink_attention_merge_launch(cudaStream_t st, const RaggedBatch& rb, const SinkAttnArgs& a) {
     if (a.nsplit > 64) return -1000;
     sink_attention_merge_kernel<<<dim3(rb.T, a.H), 128, 0, st>>>(a);
     return last_err();

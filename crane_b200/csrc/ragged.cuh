@@ -134,6 +134,14 @@ struct SinkAttnArgs {
     int v_row = 0;                           // row width of v_pool (0: dv).  kv_shared: v_row == d, a cached row's first dv columns are its value
 };
 int sink_attention_launch(cudaStream_t st, const RaggedBatch& rb, const SinkAttnArgs& a);
+// The splits' partial results joined, in split order, with the sink (what sink_attention_launch does itself when nsplit > 1)
+int sink_attention_merge_launch(cudaStream_t st, const RaggedBatch& rb, const SinkAttnArgs& a);
+// A few rows whose heads all read one key row per token (Gk == 1), bf16 pages, on the tensor cores (ragged_shared.cu): leaves the splits' partial
+// results only.  No score modifiers, no gate.  Blocks: rows x (heads / shared_key_heads(), rounded up) x nsplit, key tiles of shared_key_tile().
+int shared_key_attention_launch(cudaStream_t st, const RaggedBatch& rb, const SinkAttnArgs& a);
+bool shared_key_fits(int d, int G, int dv, bool kv_shared, bool split);
+int shared_key_heads();
+int shared_key_tile();
 
 struct Mamba2Args {
     const float* proj; int ldp;       // [T, ldp]: z | x | B | C | dt
@@ -276,8 +284,14 @@ int latent_scatter_launch(cudaStream_t st, const RaggedBatch& rb, const LatentBu
 
 // Block-diagonal linear: out[r, h * n_out + i] = sum_j in[r, h * n_in + j] * w[(h * n_in + j) * n_out + i], every product and sum in
 // f32 in the order j = 0, 1, ...  (w is stored input-major per head: [H, n_in, n_out] bf16).
-// in_w / out_w: columns from one head's slice to the next in `in` / `out` (0: n_in / n_out).
-int headwise_linear_launch(cudaStream_t st, const ActOut& in, const bf16* w, int T, int H, int n_in, int n_out, const ActOut& out, int in_w = 0, int out_w = 0);
+// in_w / out_w: columns from one head's slice to the next in `in` / `out` (0: n_in / n_out).  splits (nullable, up to headwise_few_rows() rows): the
+// input is an attention's partial results (part, nsplit, sink, dv == n_in of it), joined while they are read.
+int headwise_linear_launch(cudaStream_t st, const ActOut& in, const bf16* w, int T, int H, int n_in, int n_out, const ActOut& out, int in_w = 0, int out_w = 0,
+                           const SinkAttnArgs* splits = nullptr);
+int headwise_few_rows();
+// latent_rot_prep and the map of the queries' unrotated parts into latent space (headwise_linear with w_uk [H, dim, kv_rank]: q_out's columns 0 .. kv_rank - 1 of
+// every head), in one launch; up to headwise_few_rows() rows
+int latent_step_launch(cudaStream_t st, const RaggedBatch& rb, const LatentRotArgs& a, const bf16* w_uk);
 
 // Gated linear attention.  proj [T, ld] holds q | k | v | g | a (H*d, H*d, H*dv, H*dv, rank columns).  Per head and key channel the
 // decay is sigmoid(z)^(1 / tau), z = a2 a + b (all f32); S_t = diag(decay_t) S_(t-1) + k_t v_t^T; o_t = S_t^T (q_t * q_scale); then

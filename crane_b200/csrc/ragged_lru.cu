@@ -74,10 +74,6 @@ __global__ void __launch_bounds__(LRU_THREADS) lru_coef_kernel(RaggedBatch rb, L
     const int slot = rb.ent_slot[e], i0 = k * LRU_TOK, nt = min(LRU_TOK, rb.ent_len[e] - i0), r0 = rb.ent_row0[e] + i0, p0 = rb.ent_pos0[e] + i0;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const bf16* wt = a.w_gates + ((size_t)blk * gridDim.y + ct) * np * 2 * LRU_COLS;
-    for (int i = tid; i < LRU_TOK * LRU_COLS; i += LRU_THREADS) {
-        const int t = i / LRU_COLS, c = i % LRU_COLS;
-        so[t][c] = (t < nt && col0 + c < n) ? lru_conv(a, slot, r0 + t, i0 + t, p0 + t, cb0 + col0 + c) : 0.f;
-    }
     auto emit = [&](int t, int c, float zr, float zi, float* sa, float* sb) {      // -> the tile's decays and gated inputs, in shared memory
         float dec = 1.f, in = 0.f;
         if (t < nt && col0 + c < n) {
@@ -100,7 +96,9 @@ __global__ void __launch_bounds__(LRU_THREADS) lru_coef_kernel(RaggedBatch rb, L
             __syncthreads();
             for (int i = tid; i < LRU_TOK * sn; i += LRU_THREADS) {
                 const int t = i / sn, j = i % sn;
-                su[t * (LRU_SLAB + 1) + j] = t < nt ? lru_conv(a, slot, r0 + t, i0 + t, p0 + t, cb0 + s0 + j) : 0.f;
+                const float u = t < nt ? lru_conv(a, slot, r0 + t, i0 + t, p0 + t, cb0 + s0 + j) : 0.f;
+                su[t * (LRU_SLAB + 1) + j] = u;
+                if (s0 + j >= col0 && s0 + j < col0 + LRU_COLS) so[t][s0 + j - col0] = u;
             }
             __syncthreads();
             for (int j = 0; j < sn; ++j) {
@@ -137,8 +135,8 @@ __global__ void __launch_bounds__(LRU_THREADS) lru_coef_kernel(RaggedBatch rb, L
             // the slab of convolution outputs; a thread walks one channel down the tokens with its taps in registers where they are few
             if (const int j = tid % LRU_SLAB, tg = tid / LRU_SLAB; j < sn) {
                 constexpr int TS = LRU_TOK / (LRU_THREADS / LRU_SLAB);        // tokens per thread
-                const int t0 = tg * TS, c = cb0 + s0 + j;
-                const bool live = s0 + j < n;
+                const int t0 = tg * TS, c = cb0 + s0 + j, oc = s0 + j - col0;
+                const bool live = s0 + j < n, own = oc >= 0 && oc < LRU_COLS;
                 float w[4], h[4], bias = 0.f, xb = 0.f;
                 const bool small = a.taps <= 4;
                 if (live) { bias = a.conv_b[c]; xb = a.x_b[c]; }
@@ -162,6 +160,7 @@ __global__ void __launch_bounds__(LRU_THREADS) lru_coef_kernel(RaggedBatch rb, L
                                 h[0] = h[1]; h[1] = h[2]; h[2] = xv[q];
                             } else u = lru_conv(a, slot, r0 + t, i0 + t, p0 + t, c);
                         }
+                        if (own) so[t][oc] = u;
                         const bf16 hi = __float2bfloat16_rn(u);
                         uh[t * LRU_LDU + j] = hi; ul[t * LRU_LDU + j] = __float2bfloat16_rn(u - __bfloat162float(hi));
                     }

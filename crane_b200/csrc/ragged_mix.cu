@@ -106,22 +106,21 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(RaggedBatch rb, Latent
 // shared key part's rotation, both into the row's page; the queries' parts to where the products read them.  The row's cosines and sines
 // are taken once, in 64-bit.
 template <typename KT>
-__global__ void __launch_bounds__(256) latent_rot_prep_kernel(RaggedBatch rb, LatentRotArgs a) {
-    extern __shared__ float lcs[];                        // [rot_dims / 2] cos, then sin
-    __shared__ float red[8];
-    const int r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nrot = a.rot_dims / 2;
+__device__ __forceinline__ void latent_rot_row(const RaggedBatch& rb, const LatentRotArgs& a, int r, float* lcs) {      // lcs: [rot_dims / 2] cos, then sin
+    __shared__ float red[32];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nrot = a.rot_dims / 2, nthr = blockDim.x;
     const int e = rb.row_entry[r], pos = rb.row_pos[r], slot = rb.ent_slot[e];
     const int page = a.block_table[(size_t)slot * a.max_pages + pos / KV_PAGE];
     KT* dst = (KT*)a.pool + ((size_t)page * KV_PAGE + (pos % KV_PAGE)) * a.row_w;
     const float* q = a.proj + (size_t)r * a.ld;
     const float* low = q + (size_t)a.H * (a.dim + a.rot_dim);
-    for (int i = threadIdx.x; i < nrot; i += 256) {
+    for (int i = threadIdx.x; i < nrot; i += nthr) {
         double sn, cs;
         sincos((double)pos * a.rot_freq[i], &sn, &cs);
         lcs[i] = (float)cs; lcs[nrot + i] = (float)sn;
     }
     float ss = 0.f;
-    for (int c = threadIdx.x; c < a.kv_rank; c += 256) ss = fmaf(low[c], low[c], ss);
+    if (threadIdx.x < 256) for (int c = threadIdx.x; c < a.kv_rank; c += 256) ss = fmaf(low[c], low[c], ss);
     ss = warp_sum(ss);
     if (lane == 0) red[warp] = ss;
     __syncthreads();
@@ -129,20 +128,26 @@ __global__ void __launch_bounds__(256) latent_rot_prep_kernel(RaggedBatch rb, La
 #pragma unroll
     for (int k = 0; k < 8; ++k) tot += red[k];
     const float inv = 1.f / sqrtf(tot / (float)a.kv_rank + a.eps);
-    for (int c = threadIdx.x; c < a.kv_rank; c += 256) kv_store<KT>(dst + c, low[c] * inv * a.kv_w[c], a.kv_lo_off);
+    for (int c = threadIdx.x; c < a.kv_rank; c += nthr) kv_store<KT>(dst + c, low[c] * inv * a.kv_w[c], a.kv_lo_off);
     auto turned = [&](const float* v, int i) {            // dimension i of a rotated part
         if (i >= 2 * nrot) return v[i];
         const float cs = lcs[i >> 1], sn = lcs[nrot + (i >> 1)];
         return (i & 1) ? v[i] * cs + v[i - 1] * sn : v[i] * cs - v[i + 1] * sn;
     };
-    for (int i = threadIdx.x; i < a.rot_dim; i += 256) kv_store<KT>(dst + a.kv_rank + i, turned(low + a.kv_rank, i), a.kv_lo_off);
+    for (int i = threadIdx.x; i < a.rot_dim; i += nthr) kv_store<KT>(dst + a.kv_rank + i, turned(low + a.kv_rank, i), a.kv_lo_off);
     const int c0 = a.whole_q ? 0 : a.rot_col, n = a.q_w - c0;
-    for (int i = threadIdx.x; i < a.H * n; i += 256) {
+    for (int i = threadIdx.x; i < a.H * n; i += nthr) {
         const int h = i / n, c = c0 + i - h * n;
         const float* qh = q + (size_t)h * (a.dim + a.rot_dim);
         const float v = c < a.rot_col ? qh[c] : c < a.rot_col + a.rot_dim ? turned(qh + a.dim, c - a.rot_col) : 0.f;
         store_act(a.q_out, r, h * a.q_w + c, v);
     }
+}
+
+template <typename KT>
+__global__ void __launch_bounds__(256) latent_rot_prep_kernel(RaggedBatch rb, LatentRotArgs a) {
+    extern __shared__ float lcs[];
+    latent_rot_row<KT>(rb, a, blockIdx.x, lcs);
 }
 
 // Number i of the rows a step's queries can see -> the sequence slot and the position.
@@ -227,12 +232,40 @@ __global__ void __launch_bounds__(128) headwise_linear_kernel(ActOut in, const b
 // them, a lane owns four neighbouring columns (one 8-byte load of the bf16 weights per input row, the warp reads 256 contiguous bytes;
 // a warp's handful of rows are all requested before the first is used), and the warps' partial sums meet in warp order.
 constexpr int HWF_ROWS = 4, HWF_WARPS = 16, HWF_COLS = 128;
-__global__ void __launch_bounds__(HWF_WARPS * 32) headwise_few_kernel(ActOut in, const bf16* __restrict__ w, int T, int n_in, int n_out, ActOut out, int in_w, int out_w) {
-    extern __shared__ float hwf_s[];                      // [T][n_in] inputs, then [warps][HWF_ROWS][HWF_COLS] partial sums
+// `sp` (part != nullptr): the input rows are the partial results of an attention's splits, joined here in split order (with the sink) -- what a
+// merging kernel of its own would have stored.
+struct HeadSplits { const float* part; int nsplit, H; const float* sink; };
+__device__ __forceinline__ void headwise_few(const ActOut& in, const bf16* __restrict__ w, int T, int n_in, int n_out, const ActOut& out, int in_w, int out_w, const HeadSplits& sp,
+                                             float* hwf_s) {      // [T][n_in] inputs, then [warps][HWF_ROWS][HWF_COLS] partial sums
     float* xin = hwf_s;
     float* part = hwf_s + (((size_t)T * n_in + 3) & ~(size_t)3);
     const int h = blockIdx.y, c0 = blockIdx.x * HWF_COLS, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    for (int i = threadIdx.x; i < T * n_in; i += blockDim.x) { const int rr = i / n_in, j = i - rr * n_in; xin[i] = act_load(in, rr, h * in_w + j); }
+    if (sp.part) {
+        __shared__ float wgt[HWF_ROWS][64];
+        __shared__ float inv_l[HWF_ROWS];
+        const int ns = sp.nsplit, stride = n_in + 2;
+        if (warp < T) {                                   // a warp per row: the maximum over the splits and the sink, then each split's weight
+            const float* pp = sp.part + ((size_t)warp * sp.H + h) * ns * stride;
+            const float sink = sp.sink ? sp.sink[h] : -INFINITY;
+            const float m0 = lane < ns ? pp[(size_t)lane * stride] : -INFINITY, m1 = lane + 32 < ns ? pp[(size_t)(lane + 32) * stride] : -INFINITY;
+            const float Mx = fmaxf(warp_max(fmaxf(m0, m1)), sink);
+            const float w0 = m0 == -INFINITY ? 0.f : __expf(m0 - Mx), w1 = m1 == -INFINITY ? 0.f : __expf(m1 - Mx);
+            wgt[warp][lane] = w0; wgt[warp][lane + 32] = w1;
+            const float l0 = lane < ns ? pp[(size_t)lane * stride + 1] * w0 : 0.f, l1 = lane + 32 < ns ? pp[(size_t)(lane + 32) * stride + 1] * w1 : 0.f;
+            const float L = warp_sum(l0 + l1) + (sink == -INFINITY ? 0.f : __expf(sink - Mx));
+            if (lane == 0) inv_l[warp] = 1.f / L;
+        }
+        __syncthreads();
+        for (int i = threadIdx.x; i < T * n_in; i += blockDim.x) {
+            const int rr = i / n_in, j = i - rr * n_in;
+            const float* pp = sp.part + ((size_t)rr * sp.H + h) * ns * stride + 2 + j;
+            float o = 0.f;
+#pragma unroll 8
+            for (int s = 0; s < ns; ++s) o = fmaf(pp[(size_t)s * stride], wgt[rr][s], o);
+            xin[i] = o * inv_l[rr];
+        }
+    } else
+        for (int i = threadIdx.x; i < T * n_in; i += blockDim.x) { const int rr = i / n_in, j = i - rr * n_in; xin[i] = act_load(in, rr, h * in_w + j); }
     __syncthreads();
     const int col = c0 + 4 * lane, per = (n_in + HWF_WARPS - 1) / HWF_WARPS, j0 = warp * per, j1 = min(n_in, j0 + per);
     const bool vec = (n_out & 3) == 0;                     // (then every group of four starts on an 8-byte boundary)
@@ -274,6 +307,25 @@ __global__ void __launch_bounds__(HWF_WARPS * 32) headwise_few_kernel(ActOut in,
         for (int wq = 0; wq < HWF_WARPS; ++wq) sum += part[((size_t)wq * HWF_ROWS + rr) * HWF_COLS + c];
         store_act(out, rr, h * out_w + c0 + c, sum);
     }
+}
+
+__global__ void __launch_bounds__(HWF_WARPS * 32) headwise_few_kernel(ActOut in, const bf16* __restrict__ w, int T, int n_in, int n_out, ActOut out, int in_w, int out_w, HeadSplits sp) {
+    extern __shared__ float hwf_s[];
+    headwise_few(in, w, T, n_in, n_out, out, in_w, out_w, sp, hwf_s);
+}
+// A decode step's latent attention up to the scores: the blocks behind the last head prepare a row each (norm, rotations, page), the others map the
+// queries' unrotated parts into latent space; neither needs the other.
+template <typename KT>
+__global__ void __launch_bounds__(HWF_WARPS * 32) latent_step_kernel(RaggedBatch rb, LatentRotArgs a, const bf16* __restrict__ w_uk) {
+    extern __shared__ float hwf_s[];
+    if (blockIdx.y >= a.H) {
+        const int r = (blockIdx.y - a.H) * gridDim.x + blockIdx.x;
+        if (r < rb.T) latent_rot_row<KT>(rb, a, r, hwf_s);
+        return;
+    }
+    ActOut in;
+    in.f = const_cast<float*>(a.proj); in.ldf = a.ld;
+    headwise_few(in, w_uk, rb.T, a.dim, a.kv_rank, a.q_out, a.dim + a.rot_dim, a.q_w, HeadSplits{nullptr, 0, 0, nullptr}, hwf_s);
 }
 
 // Every entry one token: the sublayer's norm (RMS in equal groups), the convolution over the carried window and the window's shift
@@ -586,16 +638,37 @@ int latent_scatter_launch(cudaStream_t st, const RaggedBatch& rb, const LatentBu
     latent_scatter_kernel<<<n, 256, 0, st>>>(rb, a, i0);
     return last_err();
 }
-int headwise_linear_launch(cudaStream_t st, const ActOut& in, const bf16* w, int T, int H, int n_in, int n_out, const ActOut& out, int in_w, int out_w) {
+static size_t headwise_few_smem(int T, int n_in) { return ((size_t)((T * n_in + 3) & ~3) + (size_t)HWF_WARPS * HWF_ROWS * HWF_COLS) * sizeof(float); }
+int headwise_few_rows() { return HWF_ROWS; }
+int latent_step_launch(cudaStream_t st, const RaggedBatch& rb, const LatentRotArgs& a, const bf16* w_uk) {
+    if (rb.T > HWF_ROWS || a.whole_q || a.rot_col != a.kv_rank || a.kv_rank < 1 || a.rot_dim < 0 || a.rot_dims < 0 || (a.rot_dims & 1) || a.rot_dims > a.rot_dim || a.rot_dims > 4096 ||
+        a.row_w < a.kv_rank + a.rot_dim || a.q_w < a.rot_col + a.rot_dim) return -1000;
+    const int nx = (a.kv_rank + HWF_COLS - 1) / HWF_COLS;
+    const size_t sm = std::max(headwise_few_smem(rb.T, a.dim), (size_t)a.rot_dims * sizeof(float));
+    const dim3 grid(nx, a.H + (rb.T + nx - 1) / nx);
+    static SmemOptIn seen_f, seen_b;
+    if (sm > 200 * 1024) return -1000;
+    if (a.kv_f32) {
+        if (const int e = ensure_dyn_smem(latent_step_kernel<float>, sm, seen_f)) return e;
+        latent_step_kernel<float><<<grid, HWF_WARPS * 32, sm, st>>>(rb, a, w_uk);
+    } else {
+        if (const int e = ensure_dyn_smem(latent_step_kernel<bf16>, sm, seen_b)) return e;
+        latent_step_kernel<bf16><<<grid, HWF_WARPS * 32, sm, st>>>(rb, a, w_uk);
+    }
+    return last_err();
+}
+int headwise_linear_launch(cudaStream_t st, const ActOut& in, const bf16* w, int T, int H, int n_in, int n_out, const ActOut& out, int in_w, int out_w, const SinkAttnArgs* splits) {
+    if (splits && (T > HWF_ROWS || splits->nsplit > 64 || splits->dv != n_in || splits->H != H || splits->out_mult != 1.f)) return -1000;
     if (!in_w) in_w = n_in;
     if (!out_w) out_w = n_out;
     const size_t smem = (size_t)HW_ROWS * n_in * sizeof(float);
-    if ((!in.f && !in.hi) || smem > 200 * 1024) return -1000;
+    if ((!splits && !in.f && !in.hi) || smem > 200 * 1024) return -1000;
     if (T <= HWF_ROWS) {
-        const size_t sf = ((size_t)((T * n_in + 3) & ~3) + (size_t)HWF_WARPS * HWF_ROWS * HWF_COLS) * sizeof(float);
+        const size_t sf = headwise_few_smem(T, n_in);
         static SmemOptIn seen_few;
         if (const int e = ensure_dyn_smem(headwise_few_kernel, sf, seen_few)) return e;
-        headwise_few_kernel<<<dim3((n_out + HWF_COLS - 1) / HWF_COLS, H), HWF_WARPS * 32, sf, st>>>(in, w, T, n_in, n_out, out, in_w, out_w);
+        headwise_few_kernel<<<dim3((n_out + HWF_COLS - 1) / HWF_COLS, H), HWF_WARPS * 32, sf, st>>>(in, w, T, n_in, n_out, out, in_w, out_w,
+                                                                                                          splits ? HeadSplits{splits->part, splits->nsplit, H, splits->sink} : HeadSplits{nullptr, 0, 0, nullptr});
         return last_err();
     }
     static SmemOptIn seen;
