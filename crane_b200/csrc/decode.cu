@@ -38,7 +38,38 @@ __device__ __forceinline__ void cp_async16_cg(uint32_t dst, const void* src) {
 __device__ __forceinline__ void cp_async_commit_g() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_async_wait_g() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-template <int B, int EPI, bool NORM>
+// The streams' form of the staged input: a thread takes four columns of every stream at a time.  Returns its share of the sum of squares.
+template <int S>
+__device__ __forceinline__ float gemv_stage_streams(const GemvArgs& a, int b, float4* xs, int K8, bool keep) {
+    const float* x = a.fs_x + (size_t)b * S * a.K;
+    const float* y = a.fs_y + (size_t)b * a.K;
+    float* nx = a.fs_next + (size_t)b * S * a.K;
+    float ssq = 0.f;
+    for (int q = threadIdx.x; q < 2 * K8; q += GV_THREADS) {
+        const float4 yv = reinterpret_cast<const float4*>(y)[q], w = reinterpret_cast<const float4*>(a.norm_w)[q];
+        float4 xv[S], u = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int s = 0; s < S; ++s) xv[s] = reinterpret_cast<const float4*>(x + (size_t)s * a.K)[q];
+#pragma unroll
+        for (int t = 0; t < S; ++t) {
+            const float o = a.fs_w[t], c = a.fs_in[t];
+            float4 n = make_float4(o * yv.x, o * yv.y, o * yv.z, o * yv.w);
+#pragma unroll
+            for (int s = 0; s < S; ++s) {
+                const float m = a.fs_mix[s * S + t];
+                n.x = fmaf(m, xv[s].x, n.x); n.y = fmaf(m, xv[s].y, n.y); n.z = fmaf(m, xv[s].z, n.z); n.w = fmaf(m, xv[s].w, n.w);
+            }
+            u.x = fmaf(c, n.x, u.x); u.y = fmaf(c, n.y, u.y); u.z = fmaf(c, n.z, u.z); u.w = fmaf(c, n.w, u.w);
+            if (keep) reinterpret_cast<float4*>(nx + (size_t)t * a.K)[q] = n;
+        }
+        ssq = fmaf(u.x, u.x, ssq); ssq = fmaf(u.y, u.y, ssq); ssq = fmaf(u.z, u.z, ssq); ssq = fmaf(u.w, u.w, ssq);
+        xs[(size_t)(b * 2 + (q & 1)) * K8 + (q >> 1)] = make_float4(u.x * w.x, u.y * w.y, u.z * w.z, u.w * w.w);
+    }
+    return ssq;
+}
+
+// NORM: 0 the input as it is, 1 RMS norm folded in, 2 the norm of a sum of parallel streams
+template <int B, int EPI, int NORM>
 __global__ void __launch_bounds__(GV_THREADS, GV_MINB)
 gemv_kernel(GemvArgs a) {
     extern __shared__ __align__(1024) unsigned char gsm[];
@@ -90,7 +121,7 @@ gemv_kernel(GemvArgs a) {
     for (int i = tid; i < B * rpc; i += GV_THREADS) acc_s[i] = 0.f;
     // RMSNorm weights are immutable (and cold in every cache): fetch this thread's first chunk before the dependency wait
     float4 nw0 = make_float4(0.f, 0.f, 0.f, 0.f), nw1 = nw0;
-    if (NORM && tid < K8) { nw0 = reinterpret_cast<const float4*>(a.norm_w)[2 * tid]; nw1 = reinterpret_cast<const float4*>(a.norm_w)[2 * tid + 1]; }
+    if (NORM == 1 && tid < K8) { nw0 = reinterpret_cast<const float4*>(a.norm_w)[2 * tid]; nw1 = reinterpret_cast<const float4*>(a.norm_w)[2 * tid + 1]; }
 
     pdl_wait();
     pdl_launch_dependents();
@@ -99,6 +130,11 @@ gemv_kernel(GemvArgs a) {
 #pragma unroll
     for (int b = 0; b < B; ++b) {
         float ssq = 0.f;
+        if constexpr (NORM == 2) {                    // (block 0 leaves the new streams)
+            const bool keep = blockIdx.x == 0;
+            ssq = a.fs_n == 1 ? gemv_stage_streams<1>(a, b, xs, K8, keep) : a.fs_n == 2 ? gemv_stage_streams<2>(a, b, xs, K8, keep) :
+                  a.fs_n == 3 ? gemv_stage_streams<3>(a, b, xs, K8, keep) : gemv_stage_streams<4>(a, b, xs, K8, keep);
+        } else
         for (int i = tid; i < K8; i += GV_THREADS) {
             const float4* xp = reinterpret_cast<const float4*>(a.x + (size_t)b * a.ldx) + 2 * i;
             float4 lo = xp[0], hi = xp[1];
@@ -123,7 +159,8 @@ gemv_kernel(GemvArgs a) {
         }
         if (NORM) {
             const float tot = block_sum(ssq, red);
-            if (tid == 0) rstd_s[b] = rsqrtf(tot / (float)(a.norm_dim > 0 ? a.norm_dim : a.K) + a.eps);
+            const float ms = tot / (float)(a.norm_dim > 0 ? a.norm_dim : a.K) + a.eps;
+            if (tid == 0) rstd_s[b] = NORM == 2 ? 1.f / sqrtf(ms) : rsqrtf(ms);
         }
     }
     __syncthreads();
@@ -310,7 +347,7 @@ static size_t gemv_smem_bytes(int B, int K, int N, int rows_per_unit, int grid) 
     return (size_t)GV_WARPS * gv_depth(B) * GV_SEG_BYTES + (size_t)B * K * 4 + (size_t)B * rpc * 4 + 16;
 }
 
-template <int B, int EPI, bool NORM>
+template <int B, int EPI, int NORM>
 static int gemv_launch_t(cudaStream_t st, const GemvArgs& a, int num_sms, bool pdl) {
     const size_t smem = gemv_smem_bytes(B, a.K, a.N, EPI == GEMV_SILU_MUL ? 2 : 1, num_sms);
     if (smem > 227 * 1024) return -1000;
@@ -331,14 +368,18 @@ static int gemv_launch_t(cudaStream_t st, const GemvArgs& a, int num_sms, bool p
 
 template <int B>
 static int gemv_launch_b(cudaStream_t st, int epi, bool norm, const GemvArgs& a, int num_sms, bool pdl) {
+    if (norm && a.fs_x) {
+        if (a.fs_n < 1 || a.fs_n > 4 || a.fs_x == a.fs_next) return -1000;
+        return epi == GEMV_STORE ? gemv_launch_t<B, GEMV_STORE, 2>(st, a, num_sms, pdl) : epi == GEMV_RELU2 ? gemv_launch_t<B, GEMV_RELU2, 2>(st, a, num_sms, pdl) : -1000;
+    }
     switch (epi) {
         case GEMV_STORE:
-            return norm ? gemv_launch_t<B, GEMV_STORE, true>(st, a, num_sms, pdl) : gemv_launch_t<B, GEMV_STORE, false>(st, a, num_sms, pdl);
-        case GEMV_RESID: return gemv_launch_t<B, GEMV_RESID, false>(st, a, num_sms, pdl);
-        case GEMV_RELU2: return norm ? -1000 : gemv_launch_t<B, GEMV_RELU2, false>(st, a, num_sms, pdl);
+            return norm ? gemv_launch_t<B, GEMV_STORE, 1>(st, a, num_sms, pdl) : gemv_launch_t<B, GEMV_STORE, 0>(st, a, num_sms, pdl);
+        case GEMV_RESID: return gemv_launch_t<B, GEMV_RESID, 0>(st, a, num_sms, pdl);
+        case GEMV_RELU2: return norm ? -1000 : gemv_launch_t<B, GEMV_RELU2, 0>(st, a, num_sms, pdl);
         case GEMV_SILU_MUL:
-            return norm ? gemv_launch_t<B, GEMV_SILU_MUL, true>(st, a, num_sms, pdl) : gemv_launch_t<B, GEMV_SILU_MUL, false>(st, a, num_sms, pdl);
-        case GEMV_LOGITS_ARGMAX: return gemv_launch_t<B, GEMV_LOGITS_ARGMAX, true>(st, a, num_sms, pdl);
+            return norm ? gemv_launch_t<B, GEMV_SILU_MUL, 1>(st, a, num_sms, pdl) : gemv_launch_t<B, GEMV_SILU_MUL, 0>(st, a, num_sms, pdl);
+        case GEMV_LOGITS_ARGMAX: return gemv_launch_t<B, GEMV_LOGITS_ARGMAX, 1>(st, a, num_sms, pdl);
         default: return -1000;
     }
 }

@@ -65,6 +65,11 @@ struct GemvArgs {
     int ldg;
     const float* gate_bias;
     const float* bias;      // GEMV_RESID / GEMV_SILU_MUL, nullable [N]: added to W x before out_scale / before the gated unit (rows interleaved like W's)
+    // GEMV_STORE / GEMV_RELU2 with norm, nullable: the input is the RMS norm of a weighted sum of fs_n (1..4) parallel streams, which first take in
+    // a sublayer's output (ragged.cuh, StreamArgs): x'_t = sum_s fs_mix[s, t] x_s + fs_w[t] y; input = rms(sum_t fs_in[t] x'_t) norm_w.
+    // fs_x, fs_next [B, fs_n, K] (not the same buffer): the streams as they are and as they become; fs_y [B, K]
+    const float* fs_x; float* fs_next; const float* fs_y;
+    const float *fs_mix, *fs_w, *fs_in; int fs_n;
     const uint32_t* force_tokens;  // optional [out_stride]: teacher forcing -- token fed back at step s is force_tokens[s] (argmax still reported)
 };
 
@@ -98,6 +103,7 @@ struct AttnDecArgs {
 };
 
 int gemv_max_group(int K, int N, int num_sms);
+// (norm with a.fs_x set: the parallel-streams form)
 int gemv_launch(cudaStream_t st, int B, int epi, bool norm, const GemvArgs& a, int num_sms, bool pdl);
 int attn_decode_launch(cudaStream_t st, int B, int D, const AttnDecArgs& a, bool pdl);
 int embed_decode_launch(cudaStream_t st, int B, const bf16* embed, int H, const SeqState* state, float* x, bool pdl);
