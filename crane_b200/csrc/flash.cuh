@@ -37,7 +37,7 @@ flash_prefill_kernel(FlashArgs a) {
     pdl_launch_dependents();
     constexpr int BM = 64;
     constexpr int DM = D > DV ? D : DV;
-    constexpr int BN = (SPLIT || DM > 128) ? 32 : 64;     // half-page key tiles wherever a 64-key tile x 2 groups x 2 stages would not fit
+    constexpr int BN = DM > 256 ? 16 : (SPLIT || DM > 128) ? 32 : 64;     // smaller key tiles wherever a 64-key tile x 2 groups x 2 stages would not fit
     constexpr int STG = (SPLIT && DM > 128) ? 1 : 2;      // stages per group (D = 256 with hi + lo planes: one)
     constexpr int LDS = D + 8;                 // padded row (elements): conflict-free ldmatrix
     constexpr int LDV = DV + 8;
@@ -359,7 +359,7 @@ flash_prefill_kernel(FlashArgs a) {
 
 template <int D, int DV, bool CAUSAL, bool PAGED, bool SPLIT, bool RAGGED = false>
 static int flash_launch_t(cudaStream_t st, const FlashArgs& a) {
-    constexpr int P = SPLIT ? 2 : 1, GROUPS = 2, DM = D > DV ? D : DV, BN = (SPLIT || DM > 128) ? 32 : 64, STG = (SPLIT && DM > 128) ? 1 : 2;
+    constexpr int P = SPLIT ? 2 : 1, GROUPS = 2, DM = D > DV ? D : DV, BN = DM > 256 ? 16 : (SPLIT || DM > 128) ? 32 : 64, STG = (SPLIT && DM > 128) ? 1 : 2;
     constexpr int SMEM = (P * 64 * (D + 8) + GROUPS * STG * P * BN * (D + DV + 16)) * 2;
     static_assert((RAGGED ? GROUPS : 1) * STG * P * BN * (D + DV + 16) * 2 >= 128 * (DV / 2 + 4) * 4, "the merge buffer lives in group 1's ring");
     static_assert(SMEM <= 227 * 1024, "flash tile does not fit");

@@ -12,7 +12,8 @@ static int ragged_d(cudaStream_t st, const FlashArgs& a) {
     if (a.v_w <= 64) return ragged_dv<D, 64>(st, a);
     if (a.v_w <= 128) return ragged_dv<D, 128>(st, a);
     if (a.v_w <= 192) return ragged_dv<D, 192>(st, a);
-    return ragged_dv<D, 256>(st, a);
+    if constexpr (D <= 384) return ragged_dv<D, 256>(st, a);
+    return -1000;
 }
 int flash_ragged_launch(cudaStream_t st, const FlashArgs& a) {
     if (!flash_ragged_fits(a.k_w, a.v_w, a.dv) || !a.seq_len || (a.k_heads && a.nkv % a.k_heads)) return -1000;
@@ -22,7 +23,9 @@ int flash_ragged_launch(cudaStream_t st, const FlashArgs& a) {
     if (a.k_w <= 96) return ragged_d<96>(st, a);
     if (a.k_w <= 128) return ragged_d<128>(st, a);
     if (a.k_w <= 192) return ragged_d<192>(st, a);
-    return ragged_d<256>(st, a);
+    if (a.k_w <= 256) return ragged_d<256>(st, a);
+    if (a.k_w <= 384) return ragged_d<384>(st, a);
+    return ragged_d<512>(st, a);
 }
 
 }  // namespace cb

@@ -96,7 +96,9 @@ int flash_prefill_launch(cudaStream_t st, int D, bool causal, bool paged, const 
 inline bool flash_widths_fit(int D, int DV) { return (D == DV && (D == 64 || D == 128 || D == 256)) || (D == 64 && DV == 128) || (D == 128 && DV == 64); }
 // Ragged causal launches over paged caches with any widths (FlashArgs::k_w, v_w, dv): the tile is the next larger one the kernel is compiled for.
 int flash_ragged_launch(cudaStream_t st, const FlashArgs& a);
-inline bool flash_ragged_fits(int k_w, int v_w, int dv) { return k_w > 0 && k_w <= 256 && (k_w & 7) == 0 && v_w >= dv && v_w <= 256 && (v_w & 7) == 0 && dv > 0 && (dv & 1) == 0; }
+inline bool flash_ragged_fits(int k_w, int v_w, int dv) {
+    return k_w > 0 && k_w <= 512 && (k_w & 7) == 0 && v_w >= dv && v_w <= (k_w <= 384 ? 256 : 192) && (v_w & 7) == 0 && dv > 0 && (dv & 1) == 0;
+}
 int gate_mul_launch(cudaStream_t st, bf16* attn, const float* qkv, int S, int nh, int D, int q_stride, int row_width, long long lo_off = 0);
 int set_rows_launch(cudaStream_t st, float* x, int H, const int* rows, int n, const float* src, bool add);
 int cast_f32_bf16_launch(cudaStream_t st, const float* src, bf16* dst, size_t n, long long lo_off = 0);

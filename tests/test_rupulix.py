@@ -64,7 +64,7 @@ SINGLE = {
     "parallel_every_head_its_own_keys": config([layer(parallel(heads=5, kv_heads=5, dim=8, vdim=24), None)], streams=2),
     "parallel_one_key_head_unrotated": config([layer(parallel(heads=4, kv_heads=1, dim=13, vdim=21, dims=0), None)], width=66, vocab=90),
     "parallel_wide_values": config([layer(parallel(heads=2, kv_heads=1, dim=12, vdim=300), None)], width=80),
-    "parallel_keys_wider_than_the_tiles": config([layer(parallel(heads=6, kv_heads=3, dim=96, vdim=32, scale=0.1), None)], width=96),
+    "parallel_keys_wider_than_the_tiles": config([layer(parallel(heads=6, kv_heads=6, dim=96, vdim=32, scale=0.1), None)], width=96),
     "recurrence_a_block_per_channel": config([layer(parallel(right=recurrence(24, 24, 4)))], width=72, vocab=90),
     "recurrence_long_convolution": config([layer(parallel(right=recurrence(40, 2, 7)))], logit_scale=1.0),
     "recurrence_wide_blocks": config([layer(parallel(right=recurrence(420, 2, 4)), None)], width=96, vocab=100),
@@ -196,7 +196,7 @@ def test_oracle_sees_what_the_sharp_tests_are_about():
 
 # dim, rotated dimensions, vdim, rank, window of latent attention; dim, key heads, vdim of the other: widths below, at and above the tensor-core tiles' own
 TENSOR_CORE_SHAPES = [(48, 16, 64, 64, 40, 32, 2, 64), (56, 16, 48, 96, 65, 48, 2, 128), (96, 32, 128, 72, 33, 64, 3, 136), (128, 40, 96, 128, 100, 120, 2, 192),
-                      (120, 2, 200, 160, 31, 40, 1, 20), (192, 64, 256, 192, 64, 128, 2, 256)]
+                      (120, 2, 200, 160, 31, 40, 1, 20), (192, 64, 256, 192, 64, 128, 2, 256), (300, 20, 128, 64, 50, 128, 4, 192), (256, 128, 256, 64, 40, 100, 3, 248)]
 
 
 def sharp_attention(dim, rot_dim, vdim, rank, size, ldim, groups, lvdim):
