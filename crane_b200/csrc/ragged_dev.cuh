@@ -17,6 +17,19 @@ __device__ __forceinline__ void store_act(const ActOut& o, int r, int c, float v
     }
 }
 
+// four neighbouring columns at once (c and the leading dimensions multiples of 4)
+__device__ __forceinline__ void split4(const float* v, uint2& hi, uint2& lo) { split_bf16x2(v[0], v[1], hi.x, lo.x); split_bf16x2(v[2], v[3], hi.y, lo.y); }
+__device__ __forceinline__ void store_act4(const ActOut& o, int r, int c, const float* v) {
+    if (o.f) *reinterpret_cast<float4*>(o.f + (size_t)r * o.ldf + c) = make_float4(v[0], v[1], v[2], v[3]);
+    if (o.hi) {
+        uint2 hi, lo;
+        split4(v, hi, lo);
+        bf16* p = o.hi + (size_t)r * o.ldb + c;
+        *reinterpret_cast<uint2*>(p) = hi;
+        if (o.lo_off) *reinterpret_cast<uint2*>(p + o.lo_off) = lo;
+    }
+}
+
 __device__ __forceinline__ void cp_async16s(void* smem_dst, const void* gsrc) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(smem_dst)), "l"(gsrc) : "memory");
 }

@@ -136,6 +136,28 @@ __device__ __forceinline__ void latent_rot_row(const RaggedBatch& rb, const Late
     };
     for (int i = threadIdx.x; i < a.rot_dim; i += nthr) kv_store<KT>(dst + a.kv_rank + i, turned(low + a.kv_rank, i), a.kv_lo_off);
     const int c0 = a.whole_q ? 0 : a.rot_col, n = a.q_w - c0;
+    if (((c0 | n | a.dim | a.rot_dim | a.rot_col | a.q_w | a.ld | a.q_out.ldf | a.q_out.ldb) & 3) == 0) {      // four columns at a time
+        for (int i = threadIdx.x; i < a.H * (n >> 2); i += nthr) {
+            const int h = i / (n >> 2), c = c0 + 4 * (i - h * (n >> 2));
+            const float* qh = q + (size_t)h * (a.dim + a.rot_dim) + (c < a.rot_col ? c : a.dim + c - a.rot_col);
+            float v[4] = {0.f, 0.f, 0.f, 0.f};
+            if (c < a.rot_col + a.rot_dim) {
+                const float4 x = *reinterpret_cast<const float4*>(qh);
+                v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+                if (c >= a.rot_col) {
+#pragma unroll
+                    for (int p = 0; p < 4; p += 2) {
+                        const int k = (c - a.rot_col + p) >> 1;
+                        if (k >= nrot) break;
+                        const float cs = lcs[k], sn = lcs[nrot + k], u = v[p], w = v[p + 1];
+                        v[p] = u * cs - w * sn; v[p + 1] = w * cs + u * sn;
+                    }
+                }
+            }
+            store_act4(a.q_out, r, h * a.q_w + c, v);
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < a.H * n; i += nthr) {
         const int h = i / n, c = c0 + i - h * n;
         const float* qh = q + (size_t)h * (a.dim + a.rot_dim);
@@ -185,6 +207,30 @@ __global__ void __launch_bounds__(256) latent_scatter_kernel(RaggedBatch rb, Lat
         *d = h;
         if (a.out_lo) d[a.out_lo] = __float2bfloat16_rn(v - __bfloat162float(h));
     };
+    if (((a.dim | a.rot_dim | a.dv | a.k_w | a.v_w | a.ld | a.kv_rank | a.row_w) & 3) == 0) {      // four columns at a time
+        auto put4 = [&](bf16* d, const float* s) {
+            const float4 x = *reinterpret_cast<const float4*>(s);
+            const float v[4] = {x.x, x.y, x.z, x.w};
+            uint2 hi, lo;
+            split4(v, hi, lo);
+            *reinterpret_cast<uint2*>(d) = hi;
+            if (a.out_lo) *reinterpret_cast<uint2*>(d + a.out_lo) = lo;
+        };
+        for (int i = threadIdx.x; i < a.H * (kn >> 2); i += 256) {
+            const int h = i / (kn >> 2), c = 4 * (i - h * (kn >> 2));
+            bf16* d = a.k_out + (((size_t)page * a.H + h) * KV_PAGE + at) * a.k_w + c;
+            if (c < a.dim) put4(d, kv + h * a.dim + c);
+            else {
+                *reinterpret_cast<uint2*>(d) = *reinterpret_cast<const uint2*>(rot + c - a.dim);
+                if (a.out_lo) *reinterpret_cast<uint2*>(d + a.out_lo) = *reinterpret_cast<const uint2*>(rot + a.kv_lo_off + c - a.dim);
+            }
+        }
+        for (int i = threadIdx.x; i < a.H * (a.dv >> 2); i += 256) {
+            const int h = i / (a.dv >> 2), c = 4 * (i - h * (a.dv >> 2));
+            put4(a.v_out + (((size_t)page * a.H + h) * KV_PAGE + at) * a.v_w + c, kv + C + 4 * i);
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < a.H * kn; i += 256) {
         const int h = i / kn, c = i - h * kn;
         bf16* d = a.k_out + (((size_t)page * a.H + h) * KV_PAGE + at) * a.k_w + c;
